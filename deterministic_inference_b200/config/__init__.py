@@ -4,3 +4,4 @@ from .gamilorn_config import GamilornConfig
 from .zatirax_config import ZatiraxConfig
 from .kipezen_config import KipezenConfig
 from .bovitar_config import BovitarConfig
+from .nedupel_config import NedupelConfig

@@ -336,9 +336,28 @@ __device__ __forceinline__ void store_rows_qkv(unsigned src, unsigned char* stag
   }
 }
 
+// What the epilogue applies.  GATED: limit > 0: g = min(gate, limit), u = clamp(up, -limit, limit),
+// g sigmoid(alpha g) (u + 1) of the float32 sums, the sigmoid on the special-function unit like
+// silu_gate's; else silu(gate) * up.  Otherwise: squared_relu: max(z, 0)^2 of the float32 sum.
+struct Activation {
+  float limit = 0.f, alpha = 0.f;
+  int squared_relu = 0;
+};
+__device__ __forceinline__ float gate_value(float g, float u, const Activation& act) {
+  if (act.limit > 0.f) {
+    g = fminf(g, act.limit);
+    u = fminf(fmaxf(u, -act.limit), act.limit);
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(act.alpha * g * -1.4426950408889634f));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+    return g * r * (u + 1.0f);
+  }
+  return silu_gate<__nv_bfloat16>(round_to<__nv_bfloat16>(g), round_to<__nv_bfloat16>(u));
+}
+
 template <typename OutT, bool GATED, int BNL>
 __device__ __forceinline__ void store_rows(unsigned src, const CUtensorMap* map_out, unsigned char* stage,
-                                           int lane, int row0, int n0, int half) {
+                                           int lane, int row0, int n0, int half, const Activation& act) {
   constexpr int PER_BLOCK = 128 / (int)sizeof(OutT);            // output values per row of a block
   constexpr int OUT_COLS = GATED ? BNL / 2 : BNL;               // output columns of a tile
   // a gated tile of 64 + 64 rows has one block of output columns: the first half's warps take it
@@ -364,8 +383,7 @@ __device__ __forceinline__ void store_rows(unsigned src, const CUtensorMap* map_
           float y[8];
 #pragma unroll
           for (int e = 0; e < 8; ++e)
-            y[e] = silu_gate<__nv_bfloat16>(round_to<__nv_bfloat16>(__uint_as_float(g[q * 8 + e])),
-                                            round_to<__nv_bfloat16>(__uint_as_float(u[q * 8 + e])));
+            y[e] = gate_value(__uint_as_float(g[q * 8 + e]), __uint_as_float(u[q * 8 + e]), act);
           stage_piece(stage, lane, h * 4 + q,
                       make_uint4(pack2_bf16(y[0], y[1]), pack2_bf16(y[2], y[3]), pack2_bf16(y[4], y[5]),
                                  pack2_bf16(y[6], y[7])));
@@ -377,6 +395,13 @@ __device__ __forceinline__ void store_rows(unsigned src, const CUtensorMap* map_
         unsigned v[32];
         tc_ld32(src + col + h * 32, v);
         tc_wait_ld();
+        if (act.squared_relu) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) {
+            const float z = fmaxf(__uint_as_float(v[e]), 0.f);
+            v[e] = __float_as_uint(z * z);
+          }
+        }
 #pragma unroll
         for (int q = 0; q < 4; ++q)
           stage_piece(stage, lane, h * 4 + q,
@@ -408,7 +433,8 @@ template <typename OutT, bool GATED, int BNL, bool QKV = false>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_large_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                   const __grid_constant__ CUtensorMap map_out, int M, int N, int K, int m_tiles_given, int n_tiles,
-                  const __grid_constant__ QkvEpilogue qk, const int* __restrict__ tile_matrix, int matrix_rows) {
+                  const __grid_constant__ QkvEpilogue qk, const int* __restrict__ tile_matrix, int matrix_rows,
+                  const __grid_constant__ Activation act) {
   // GROUPED (tile_matrix not null): the weights are a stack of matrices of matrix_rows rows each, and
   // the token tile m multiplies matrix tile_matrix[m] (a negative entry: matrix 0, for a tile of
   // padding whose result nobody reads).  The table is written by the kernel before this one, and the
@@ -562,7 +588,7 @@ gemm_large_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
                          rows, &map_out, m0 + quarter * 32);
       } else {
         store_rows<OutT, GATED, BNL>(tmem + buf * BNL + lane_base, &map_out, epi_stage + (warp - EPI_WARP0) * EPI_STAGE_BYTES,
-                                     lane, m0 + quarter * 32, n0, half);
+                                     lane, m0 + quarter * 32, n0, half, act);
       }
       tc_fence_before();
       __syncwarp();
@@ -653,7 +679,7 @@ template <typename OutT, bool GATED, int BNL, bool QKV = false>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                  const __grid_constant__ CUtensorMap map_out, int M, int N, int K, int m_tiles, int n_tiles,
-                 const __grid_constant__ QkvEpilogue qk) {
+                 const __grid_constant__ QkvEpilogue qk, const __grid_constant__ Activation act) {
   static_assert(!GATED || BNL == 256, "the gated epilogue pairs 128 gate rows with 128 up rows");
   using TL = PairTile<BNL, QKV>;
   constexpr int STAGE_BYTES = TL::STAGE_BYTES, STAGES = TL::STAGES;
@@ -786,7 +812,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
                        &map_out, m0 + quarter * 32);
       else
         store_rows<OutT, GATED, BNL>(tmem + buf * BNL + lane_base, &map_out, epi_stage + (warp - EPI_WARP0) * EPI_STAGE_BYTES,
-                                     lane, m0 + quarter * 32, n0, half);
+                                     lane, m0 + quarter * 32, n0, half, act);
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive_cluster(acc_empty0 + buf * 8);
@@ -853,7 +879,7 @@ bool make_out_map(CUtensorMap* map, void* ptr, long long M, long long N) {
 template <typename OutT, bool GATED, int BNL, bool QKV = false>
 int launch_large(const void* x, const void* w, void* out, int M, int N, int K, int sm_count,
                  cudaStream_t st, const QkvEpilogue& qk = QkvEpilogue{}, const int* tile_matrix = nullptr,
-                 int matrices = 1) {
+                 int matrices = 1, const Activation& act = Activation{}) {
   CUtensorMap mx, mw, mo;
   const long long matrix_rows = GATED ? 2ll * N : (long long)N;
   if (!make_map(&mx, x, M, K, BM) || !make_map(&mw, w, matrices * matrix_rows, K, GATED ? BNL / 2 : 128) ||
@@ -874,14 +900,14 @@ int launch_large(const void* x, const void* w, void* out, int M, int N, int K, i
   }
   const int grid = (int)(tiles < sm_count ? tiles : sm_count);
   dib_launch(kern, dim3(grid), dim3(THREADS), SMEM_BYTES, st, mx, mw, mo, M, N, K, m_tiles, n_tiles, qk, tile_matrix,
-             (int)matrix_rows);
+             (int)matrix_rows, act);
   DIB_CHECK_LAUNCH();
   return DIB_OK;
 }
 
 template <typename OutT, bool GATED, int BNL, bool QKV = false>
 int launch_pair(const void* x, const void* w, void* out, int M, int N, int K, int sm_count,
-                cudaStream_t st, const QkvEpilogue& qk = QkvEpilogue{}) {
+                cudaStream_t st, const QkvEpilogue& qk = QkvEpilogue{}, const Activation& act = Activation{}) {
   CUtensorMap mx, mw, mo;
   if (!make_map(&mx, x, M, K, BM) || !make_map(&mw, w, GATED ? 2ll * N : (long long)N, K, BNL / 2) ||
       !make_out_map<OutT>(&mo, out, M, QKV ? (long long)qk.Hq * 128 : (long long)N))
@@ -914,7 +940,7 @@ int launch_pair(const void* x, const void* w, void* out, int M, int N, int K, in
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = dib_pdl_enabled() ? 2 : 1;
-  cudaLaunchKernelEx(&cfg, kern, mx, mw, mo, M, N, K, m_tiles, n_tiles, qk);
+  cudaLaunchKernelEx(&cfg, kern, mx, mw, mo, M, N, K, m_tiles, n_tiles, qk, act);
   DIB_CHECK_LAUNCH();
   return DIB_OK;
 }
@@ -974,6 +1000,21 @@ int dib_gemm_bf16_large(const void* x, const void* w, void* out, int M, int N, i
   return launch_large<__nv_bfloat16, false, 256>(x, w, out, M, N, K, sm_count, st);
 }
 
+// out[M, N] = max(x w^T, 0)^2, bfloat16, the square of the float32 sum.  K and N multiples of 8.
+int dib_gemm_bf16_large_squared_relu(const void* x, const void* w, void* out, int M, int N, int K, int sm_count,
+                                     cudaStream_t st) {
+  if (M == 0 || N == 0) return DIB_OK;
+  if (K < 8 || K % 8 != 0 || sm_count < 1 || N % 8 != 0) return DIB_BAD_SIZE;
+  if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) % 16 != 0)
+    return DIB_BAD_ALIGN;
+  Activation act;
+  act.squared_relu = 1;
+  const int shape = tile_shape(M, N, sm_count);
+  if (shape == 2) return launch_pair<__nv_bfloat16, false, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, act);
+  if (shape == 0) return launch_large<__nv_bfloat16, false, 128>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, nullptr, 1, act);
+  return launch_large<__nv_bfloat16, false, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, nullptr, 1, act);
+}
+
 // out[M, I] = silu(x w_gate^T) * (x w_up^T) with w = [w_gate ; w_up] of shape [2I, K]; bf16 in
 // and out.  I a multiple of 8, K of 8.
 int dib_gemm_bf16_large_gated(const void* x, const void* w, void* out, int M, int I, int K,
@@ -991,18 +1032,22 @@ int dib_gemm_bf16_large_gated(const void* x, const void* w, void* out, int M, in
 // A product per tile of 128 rows with one of a stack of matrices: row tile m of x [M, K] (M a multiple
 // of 128) times matrix tile_matrix[m] of w.  gated = 0: w [matrices, N, K], out [M, N] bfloat16 or
 // float32 (N a multiple of 256).  gated = 1: w [matrices, 2N, K] (gate rows, then up rows), out [M, N]
-// bfloat16 = silu(gate) * up (N a multiple of 128).  The table lies on the device and may be written
+// bfloat16 = silu(gate) * up, or with limit > 0 the limited gate of gate_value (N a multiple of 128).  The table lies on the device and may be written
 // by the kernel before this one; it has M / 128 entries and one more, the number of row tiles in use
 // (the first ones; the rows of the others are left as they are).  Tiles of 128 x 256 by one CTA.
 int dib_gemm_bf16_large_grouped(const void* x, const void* w, void* out, int M, int N, int K, int gated, int out_fp32,
-                                const int* tile_matrix, int matrices, int sm_count, cudaStream_t st) {
+                                const int* tile_matrix, int matrices, float limit, float alpha, int sm_count,
+                                cudaStream_t st) {
   if (M == 0 || N == 0) return DIB_OK;
   if (K < 8 || K % 8 != 0 || sm_count < 1 || M % BM != 0 || matrices < 1 || tile_matrix == nullptr ||
       N % (gated ? 128 : 256) != 0 || (gated && out_fp32))
     return DIB_BAD_SIZE;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) % 16 != 0)
     return DIB_BAD_ALIGN;
-  if (gated) return launch_large<__nv_bfloat16, true, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, tile_matrix, matrices);
+  Activation act;
+  act.limit = limit;
+  act.alpha = alpha;
+  if (gated) return launch_large<__nv_bfloat16, true, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, tile_matrix, matrices, act);
   if (out_fp32) return launch_large<float, false, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, tile_matrix, matrices);
   return launch_large<__nv_bfloat16, false, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, tile_matrix, matrices);
 }

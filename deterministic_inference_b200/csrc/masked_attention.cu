@@ -217,12 +217,16 @@ attn_prepare_row_kernel(Source proj, long long row_width, const float* __restric
 // rotates the key part into its last R; slot 1 + h rotates the last R elements of query head h into
 // q_out[t, h, C .. C + R) (the first C are the product of the head's other Dn elements with its
 // key map, written by the per-head product).  The cache row of a token is [C + R], one key head.
+// The rotation pairs element i with i + R/2 (pairs == 0) or element 2i with 2i + 1 (pairs == 1);
+// cosine and sine are multiplied by `amp`.  cache null: nothing is stored, and the row may be the query
+// heads alone (a layer that reads another layer's rows).
 template <typename T>
 __global__ void __launch_bounds__(WARPS * 32)
 latent_prepare_kernel(Source proj, long long row_width, T* __restrict__ q_out, T* __restrict__ cache,
                       const float* __restrict__ c_w, float eps, const float* __restrict__ freq,
                       const int* __restrict__ positions, const int* __restrict__ slot_mapping,
-                      int T_tokens, int H, int Dn, int R, int C, int page_size, long long num_pages) {
+                      int T_tokens, int H, int Dn, int R, int C, int page_size, long long num_pages, int pairs,
+                      float amp) {
   pdl_prologue(proj.p);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int slots = H + 1;
@@ -255,12 +259,12 @@ latent_prepare_kernel(Source proj, long long row_width, T* __restrict__ q_out, T
     dst = q_out + ((long long)t * H + (s - 1)) * (C + R) + C;
   }
   for (int d = lane; d < R; d += 32) {
-    const int i = d < half ? d : d - half;
-    const float a = __fmul_rn(pos, freq[i]);
-    const float c = cosf(a), sn = sinf(a);
+    const bool first = pairs ? (d & 1) == 0 : d < half;
+    const float a = __fmul_rn(pos, freq[pairs ? d >> 1 : (first ? d : d - half)]);
+    const float c = __fmul_rn(amp, cosf(a)), sn = __fmul_rn(amp, sinf(a));
     const float u = round_to<T>(source_load(proj, src + d));
-    const float o = round_to<T>(source_load(proj, src + (d < half ? d + half : d - half)));
-    Elem<T>::store(dst + d, d < half ? __fmaf_rn(u, c, -__fmul_rn(o, sn)) : __fmaf_rn(u, c, __fmul_rn(o, sn)));
+    const float o = round_to<T>(source_load(proj, src + (pairs ? (d ^ 1) : (first ? d + half : d - half))));
+    Elem<T>::store(dst + d, first ? __fmaf_rn(u, c, -__fmul_rn(o, sn)) : __fmaf_rn(u, c, __fmul_rn(o, sn)));
   }
 }
 
@@ -517,19 +521,20 @@ int dib_attn_prepare_row(const void* proj, int kind, int splits, long long strid
 int dib_latent_prepare(const void* proj, int kind, int splits, long long stride, long long row_width, void* q_out,
                        void* cache, const float* c_w, float eps, const float* freq, const int* positions,
                        const int* slot_mapping, int T, int H, int Dn, int R, int C, int page_size,
-                       long long num_pages, int dtype, cudaStream_t st) {
+                       long long num_pages, int dtype, int pairs, float amp, cudaStream_t st) {
   if (T == 0) return DIB_OK;
-  if (H < 1 || Dn < 1 || R < 2 || R % 2 || C < 1 || page_size < 1 || freq == nullptr || c_w == nullptr)
+  if (H < 1 || Dn < 1 || R < 2 || R % 2 || C < 1 || page_size < 1 || freq == nullptr ||
+      (cache != nullptr && (c_w == nullptr || row_width < (long long)H * (Dn + R) + C + R)) || row_width < (long long)H * (Dn + R))
     return DIB_BAD_SIZE;
   const Source src = make_source(proj, kind, splits, stride);
   const int blocks = ceil_div_host((long long)T * (H + 1), WARPS);
   if (dtype == 0)
     dib_launch(latent_prepare_kernel<float>, dim3(blocks), dim3(WARPS * 32), 0, st, src, row_width, (float*)q_out,
-               (float*)cache, c_w, eps, freq, positions, slot_mapping, T, H, Dn, R, C, page_size, num_pages);
+               (float*)cache, c_w, eps, freq, positions, slot_mapping, T, H, Dn, R, C, page_size, num_pages, pairs, amp);
   else if (dtype == 1)
     dib_launch(latent_prepare_kernel<__nv_bfloat16>, dim3(blocks), dim3(WARPS * 32), 0, st, src, row_width,
                (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, c_w, eps, freq, positions, slot_mapping, T, H, Dn, R,
-               C, page_size, num_pages);
+               C, page_size, num_pages, pairs, amp);
   else return DIB_BAD_DTYPE;
   DIB_CHECK_LAUNCH();
   return DIB_OK;

@@ -6,11 +6,14 @@
 //             2) largest choice scores, the best `group_keep` groups stay; of their experts the `top`
 //             largest choice scores win (ties: the lower index); weight_j = s_j / (sum of the chosen
 //             s + eps) * scale, or s_j * scale (normalize 0).  One warp per token, float32.
+//             A table of choices [V][top] (the experts of a token id) takes the route's place: the sort
+//             reads it by the step's token ids, and every weight is one constant.
 //   sort:     pairs p = t * top + j are placed, by expert, into tiles of `tile` rows; an expert's
 //             rows are filled up to whole tiles (row -> pair or -1; tile -> expert or -1).
-//   gate/up:  hidden[row] = silu(x[token] Wg_e^T) * (x[token] Wu_e^T), rounded once to x's type.
+//   gate/up:  hidden[row] = act(x[token] Wg_e^T, x[token] Wu_e^T), rounded once to x's type; act(g, u) =
+//             silu(g) u, or, limited, min(g, l) sigmoid(alpha min(g, l)) (clamp(u, -l, l) + 1).
 //   down:     per_pair[pair] = hidden[row] Wd_e^T, float32.
-//   combine:  out[t] = sum_j weight[t, j] per_pair[t * top + j] (in the order of j)
+//   combine:  out[t] = sum_j weight[t, j] (or the constant) per_pair[t * top + j] (in the order of j)
 //                      + sigmoid(logits[t, col]) * shared[t] (col < 0: + shared[t]).
 //
 // A row's sums never depend on the other rows of its tile, on the tile's size or on where the row
@@ -136,15 +139,23 @@ moe_route_kernel(Source logits, long long row_width, const float* __restrict__ c
 // One block.  Where a pair lands inside its expert's rows depends on the order in which threads arrive,
 // which no result depends on (a row's sums do not know the row's place).
 constexpr int SORT_THREADS = 1024;
+// table given: ids are the step's token ids and pair i's expert is table[ids[i / top]][i % top]
+// (a token id outside the table takes its nearest row, as the embedding does).
 __global__ void __launch_bounds__(SORT_THREADS)
-moe_sort_kernel(const int* __restrict__ ids, int pairs, int E, int tile, int max_tiles, int* __restrict__ order) {
+moe_sort_kernel(const int* ids, const int* __restrict__ table, int top, int V, int pairs, int E, int tile, int max_tiles,
+                int* __restrict__ order) {
   __shared__ int count[SORT_THREADS], first_tile[SORT_THREADS + 1], scan[SORT_THREADS];
   pdl_prologue(ids);
   const int e = threadIdx.x;
+  auto expert_of = [&](int i) {
+    if (table == nullptr) return ids[i];
+    const int t = i / top, id = ids[t] < 0 ? 0 : (ids[t] >= V ? V - 1 : ids[t]);
+    return table[(long long)id * top + i - t * top];
+  };
   count[e] = 0;
   __syncthreads();
   for (int i = threadIdx.x; i < pairs; i += SORT_THREADS) {
-    const int x = ids[i];
+    const int x = expert_of(i);
     if (x >= 0 && x < E) atomicAdd(&count[x], 1);
   }
   __syncthreads();
@@ -169,7 +180,7 @@ moe_sort_kernel(const int* __restrict__ ids, int pairs, int E, int tile, int max
     for (int k = first_tile[e]; k < first_tile[e + 1] && k < max_tiles; ++k) tile_expert[k] = e;
   if (e == 0) tile_expert[max_tiles] = first_tile[E] < max_tiles ? first_tile[E] : max_tiles;   // tiles in use: the first ones
   for (int i = threadIdx.x; i < pairs; i += SORT_THREADS) {
-    const int x = ids[i];
+    const int x = expert_of(i);
     if (x < 0 || x >= E) continue;
     const long long at = (long long)first_tile[x] * tile + atomicAdd(&count[x], 1);
     if (at < (long long)max_tiles * tile) order[at] = i;
@@ -178,8 +189,18 @@ moe_sort_kernel(const int* __restrict__ ids, int pairs, int E, int tile, int max
 
 // ---- the grouped products -------------------------------------------------------------------------
 // mode 0 (gate and up): A row r = x[pair / top] (K = the model's width), B = the expert's [2F][K] (gate
-// rows, then up rows), out hidden[row][F] = silu(gate) * up in T.
+// rows, then up rows), out hidden[row][F] = act(gate, up) in T.
 // mode 1 (down): A row r = hidden[row] (K = F), B = the expert's [N][K], out per_pair[pair][N] float32.
+
+// limit > 0: the limited gate; else silu
+__device__ __forceinline__ float expert_gate(float g, float u, float limit, float alpha) {
+  if (limit > 0.f) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * sigmoid_f32(alpha * g) * (u + 1.0f);
+  }
+  return g * sigmoid_f32(g) * u;
+}
 
 __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3,
                                                unsigned b0, unsigned b1) {
@@ -200,7 +221,7 @@ template <int MT, int NJ>
 __global__ void __launch_bounds__(GP_THREADS)
 moe_product_mma_kernel(const __nv_bfloat16* __restrict__ a_rows, const int* __restrict__ order, int max_tiles,
                        int tile, int top, const __nv_bfloat16* __restrict__ w, void* out, int K, int N, int KC,
-                       int mode) {
+                       int mode, float limit, float alpha) {
   extern __shared__ __align__(16) unsigned char gp_smem[];
   __nv_bfloat16* As = reinterpret_cast<__nv_bfloat16*>(gp_smem);     // [MT * 16][KC + GP_PAD]
   __shared__ int row_pair[MT * 16];
@@ -283,7 +304,7 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ a_rows, const int* __re
           for (int e = 0; e < 2; ++e) {
             const int n = n0 + j * 8 + tig * 2 + e;
             const float gt = acc[m][j][2 * hh + e], up = acc[m][j + NJ / 2][2 * hh + e];
-            if (n < N) dst[n] = __float2bfloat16_rn(gt * sigmoid_f32(gt) * up);
+            if (n < N) dst[n] = __float2bfloat16_rn(expert_gate(gt, up, limit, alpha));
           }
       } else {
         float* dst = reinterpret_cast<float*>(out) + (long long)pair * N;
@@ -304,7 +325,7 @@ constexpr int GC_ROWS = 16, GC_COLS = 128, GC_K = 128;
 template <typename T>
 __global__ void __launch_bounds__(GC_COLS)
 moe_product_kernel(const T* __restrict__ a_rows, const int* __restrict__ order, int max_tiles, int tile, int top,
-                   const T* __restrict__ w, void* out, int K, int N, int mode) {
+                   const T* __restrict__ w, void* out, int K, int N, int mode, float limit, float alpha) {
   __shared__ float xs[GC_ROWS][GC_K];
   __shared__ int row_pair[GC_ROWS];
   pdl_prologue(a_rows, order);
@@ -354,23 +375,23 @@ moe_product_kernel(const T* __restrict__ a_rows, const int* __restrict__ order, 
     if (pair < 0) continue;
     if (mode == 0)
       Elem<T>::store(reinterpret_cast<T*>(out) + ((long long)tl * tile + r0 + r) * N + n,
-                     acc0[r] * sigmoid_f32(acc0[r]) * acc1[r]);
+                     expert_gate(acc0[r], acc1[r], limit, alpha));
     else
       reinterpret_cast<float*>(out)[(long long)pair * N + n] = acc0[r];
   }
 }
 
 // out[t, c] = sum_j weights[t, j] * per_pair[t * top + j, c], j ascending, + sigmoid(gate[t]) * shared[t, c]
-// (gate_col < 0: the shared expert has no gate and is added as it is)
-__global__ void moe_combine_kernel(const float* __restrict__ per_pair, const float* __restrict__ weights, Source shared,
-                                   Source logits, long long logit_row, int gate_col, float* __restrict__ out, int T,
+// (gate_col < 0: the shared expert has no gate and is added as it is; weights null: every weight is `weight`)
+__global__ void moe_combine_kernel(const float* __restrict__ per_pair, const float* __restrict__ weights, float weight,
+                                   Source shared, Source logits, long long logit_row, int gate_col, float* __restrict__ out, int T,
                                    int top, int W) {
   pdl_prologue(per_pair, weights, shared.p, logits.p);
   const long long n = (long long)T * W;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const long long t = i / W, c = i - t * W;
     float v = 0.f;
-    for (int j = 0; j < top; ++j) v = __fmaf_rn(weights[t * top + j], per_pair[(t * top + j) * W + c], v);
+    for (int j = 0; j < top; ++j) v = __fmaf_rn(weights != nullptr ? weights[t * top + j] : weight, per_pair[(t * top + j) * W + c], v);
     if (shared.p != nullptr)
       v = gate_col < 0 ? __fadd_rn(v, source_load(shared, i))
                        : __fmaf_rn(sigmoid_f32(source_load(logits, t * logit_row + gate_col)), source_load(shared, i), v);
@@ -380,7 +401,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ per_pair, const flo
 
 template <int MT, int NJ>
 int launch_product_mma(const void* a_rows, const int* order, int max_tiles, int tile, int top, const void* w, void* out,
-                       int K, int N, int mode, cudaStream_t st) {
+                       int K, int N, int mode, float limit, float alpha, cudaStream_t st) {
   // the A rows' k are staged in runs of KC (a multiple of 64) that fit 64 KB; tiles of 16 rows (decoded
   // tokens: the product is bound by how many weight loads an SM keeps in flight) in runs that fit 16 KB,
   // so that an SM holds many CTAs.  The runs do not change the order of a sum.
@@ -396,27 +417,27 @@ int launch_product_mma(const void* a_rows, const int* order, int max_tiles, int 
   }
   const int per_cta = mode == 0 ? 16 * NJ : 32 * NJ;
   dib_launch(moe_product_mma_kernel<MT, NJ>, dim3(max_tiles, (N + per_cta - 1) / per_cta), dim3(GP_THREADS), smem, st,
-             (const __nv_bfloat16*)a_rows, order, max_tiles, tile, top, (const __nv_bfloat16*)w, out, K, N, KC, mode);
+             (const __nv_bfloat16*)a_rows, order, max_tiles, tile, top, (const __nv_bfloat16*)w, out, K, N, KC, mode, limit, alpha);
   DIB_CHECK_LAUNCH();
   return DIB_OK;
 }
 
 // mode 0: gate and up; 1: down.  dtype 0 float32, 1 bfloat16.
 int moe_product(const void* a_rows, int dtype, const int* order, int max_tiles, int tile, int top, const void* w,
-                void* out, int K, int N, int mode, cudaStream_t st) {
+                void* out, int K, int N, int mode, float limit, float alpha, cudaStream_t st) {
   if (max_tiles == 0) return DIB_OK;
   if (K < 1 || N < 1 || tile < 1 || tile % GC_ROWS || top < 1) return DIB_BAD_SIZE;
   if (dtype == 1 && K % 8 == 0 && (tile == 16 || tile == 64)) {
-    if (tile == 16) return launch_product_mma<1, 4>(a_rows, order, max_tiles, tile, top, w, out, K, N, mode, st);
-    return launch_product_mma<4, 4>(a_rows, order, max_tiles, tile, top, w, out, K, N, mode, st);
+    if (tile == 16) return launch_product_mma<1, 4>(a_rows, order, max_tiles, tile, top, w, out, K, N, mode, limit, alpha, st);
+    return launch_product_mma<4, 4>(a_rows, order, max_tiles, tile, top, w, out, K, N, mode, limit, alpha, st);
   }
   const dim3 grid(max_tiles, (N + GC_COLS - 1) / GC_COLS, tile / GC_ROWS);
   if (dtype == 0)
     dib_launch(moe_product_kernel<float>, grid, dim3(GC_COLS), 0, st, (const float*)a_rows, order, max_tiles, tile, top,
-               (const float*)w, out, K, N, mode);
+               (const float*)w, out, K, N, mode, limit, alpha);
   else if (dtype == 1)
     dib_launch(moe_product_kernel<__nv_bfloat16>, grid, dim3(GC_COLS), 0, st, (const __nv_bfloat16*)a_rows, order,
-               max_tiles, tile, top, (const __nv_bfloat16*)w, out, K, N, mode);
+               max_tiles, tile, top, (const __nv_bfloat16*)w, out, K, N, mode, limit, alpha);
   else return DIB_BAD_DTYPE;
   DIB_CHECK_LAUNCH();
   return DIB_OK;
@@ -492,34 +513,37 @@ int dib_moe_route(const void* logits, int kind, int splits, long long stride, lo
   return DIB_OK;
 }
 
-// order: int32 [max_tiles * tile + max_tiles + 1]; max_tiles >= pairs / tile + min(E, pairs)
-int dib_moe_sort(const int* ids, int pairs, int E, int tile, int max_tiles, int* order, cudaStream_t st) {
+// order: int32 [max_tiles * tile + max_tiles + 1]; max_tiles >= pairs / tile + min(E, pairs).  table null: ids
+// [pairs] are experts; else ids [pairs / top] are token ids, whose experts table [V][top] gives.
+int dib_moe_sort(const int* ids, const int* table, int top, int V, int pairs, int E, int tile, int max_tiles, int* order,
+                 cudaStream_t st) {
   if (pairs == 0) return DIB_OK;
-  if (E < 1 || E > SORT_THREADS || tile < 1 || max_tiles < 1) return DIB_BAD_SIZE;
-  dib_launch(moe_sort_kernel, dim3(1), dim3(SORT_THREADS), 0, st, ids, pairs, E, tile, max_tiles, order);
+  if (E < 1 || E > SORT_THREADS || tile < 1 || max_tiles < 1 || (table != nullptr && (top < 1 || V < 1))) return DIB_BAD_SIZE;
+  dib_launch(moe_sort_kernel, dim3(1), dim3(SORT_THREADS), 0, st, ids, table, top, V, pairs, E, tile, max_tiles, order);
   DIB_CHECK_LAUNCH();
   return DIB_OK;
 }
 
+// limit > 0: the limited gate (limit, alpha); else silu
 int dib_moe_gate_up(const void* x, int dtype, const int* order, int max_tiles, int tile, int top, const void* w_gate_up,
-                    void* hidden, int F, int W, cudaStream_t st) {
-  return moe_product(x, dtype, order, max_tiles, tile, top, w_gate_up, hidden, W, F, 0, st);
+                    void* hidden, int F, int W, float limit, float alpha, cudaStream_t st) {
+  return moe_product(x, dtype, order, max_tiles, tile, top, w_gate_up, hidden, W, F, 0, limit, alpha, st);
 }
 
 int dib_moe_down(const void* hidden, int dtype, const int* order, int max_tiles, int tile, const void* w_down,
                  float* per_pair, int F, int W, cudaStream_t st) {
-  return moe_product(hidden, dtype, order, max_tiles, tile, 1, w_down, per_pair, F, W, 1, st);
+  return moe_product(hidden, dtype, order, max_tiles, tile, 1, w_down, per_pair, F, W, 1, 0.f, 0.f, st);
 }
 
-// shared null: no shared expert.
-int dib_moe_combine(const float* per_pair, const float* weights, const void* shared, int skind, int ssplits,
+// shared null: no shared expert.  weights null: every weight is `weight`.
+int dib_moe_combine(const float* per_pair, const float* weights, float weight, const void* shared, int skind, int ssplits,
                     long long sstride, const void* logits, int lkind, int lsplits, long long lstride,
                     long long logit_row, int gate_col, float* out, int T, int top, int W, cudaStream_t st) {
   if (T == 0) return DIB_OK;
   if (top < 1 || W < 1) return DIB_BAD_SIZE;
   const long long n = (long long)T * W;
   const int blocks = (int)((n + 255) / 256 > 148 * 16 ? 148 * 16 : (n + 255) / 256);
-  dib_launch(moe_combine_kernel, dim3(blocks), dim3(256), 0, st, per_pair, weights,
+  dib_launch(moe_combine_kernel, dim3(blocks), dim3(256), 0, st, per_pair, weights, weight,
              make_source(shared, skind, ssplits, sstride), make_source(logits, lkind, lsplits, lstride), logit_row,
              gate_col, out, T, top, W);
   DIB_CHECK_LAUNCH();

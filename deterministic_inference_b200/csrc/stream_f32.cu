@@ -227,6 +227,16 @@ __global__ void xielu_kernel(Source z, float ap, float an, void* out, int out_dt
   }
 }
 
+// out = max(z, 0)^2
+__global__ void squared_relu_kernel(Source z, void* out, int out_dtype, long long n) {
+  pdl_prologue(z.p);
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n;
+       i += (long long)gridDim.x * blockDim.x) {
+    const float x = fmaxf(source_load(z, i), 0.f);
+    store_as(out, out_dtype, i, x * x);
+  }
+}
+
 // x = cap * tanh(x / cap), in place
 __global__ void softcap_kernel(float* x, float cap, long long n) {
   pdl_prologue();
@@ -357,6 +367,16 @@ int dib_xielu(const void* z, int kind, int splits, long long stride, float ap, f
   if (out_dtype != 0 && out_dtype != 1) return DIB_BAD_DTYPE;
   dib_launch(xielu_kernel, dim3(flat_grid(n, 256)), dim3(256), 0, st, make_source(z, kind, splits, stride), ap,
              an, out, out_dtype, n);
+  DIB_CHECK_LAUNCH();
+  return DIB_OK;
+}
+
+int dib_squared_relu(const void* z, int kind, int splits, long long stride, void* out, int out_dtype, long long n,
+                     cudaStream_t st) {
+  if (n == 0) return DIB_OK;
+  if (out_dtype != 0 && out_dtype != 1) return DIB_BAD_DTYPE;
+  dib_launch(squared_relu_kernel, dim3(flat_grid(n, 256)), dim3(256), 0, st, make_source(z, kind, splits, stride), out,
+             out_dtype, n);
   DIB_CHECK_LAUNCH();
   return DIB_OK;
 }

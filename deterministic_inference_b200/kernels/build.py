@@ -18,6 +18,7 @@ from __future__ import annotations
 import ctypes
 import hashlib
 import os
+import re
 import shutil
 import subprocess
 import sys
@@ -46,6 +47,7 @@ SOURCES = {
     "linear_recurrence": "linear_recurrence.cu",
     "routed_experts": "routed_experts.cu",
     "state_space": "state_space.cu",
+    "retention": "retention.cu",
 }
 HEADERS = ("common.cuh", "attention_merge.cuh")
 # further headers a library includes
@@ -60,6 +62,7 @@ EXTRA_HEADERS = {
     "state_space": ("source.cuh", "conv_tail.cuh"),
     "linear_recurrence": ("source.cuh", "conv_tail.cuh"),
     "routed_experts": ("source.cuh",),
+    "retention": ("source.cuh", "sigmoid_attention_mma.cuh"),
 }
 
 NVCC_FLAGS = [
@@ -184,8 +187,10 @@ def compile_library(name: str, verbose: bool = True) -> Path:
         tmp.unlink(missing_ok=True)
         raise KernelBuildError(f"nvcc failed for {SOURCES[name]}:\n{' '.join(cmd)}\n{log}")
     os.replace(tmp, out)
+    # older builds of this library (its name and a hash: "gemm_bf16" is not "gemm_bf16_large")
+    stale = re.compile(rf"libdib200_{re.escape(name)}_[0-9a-f]+\.so")
     for old in out.parent.glob(f"libdib200_{name}_*.so"):
-        if old != out and ".tmp" not in old.name:
+        if old != out and stale.fullmatch(old.name):
             old.unlink(missing_ok=True)
     if verbose:
         print(f"[dib200] built {out.name} in {time.time() - t0:.1f} s", file=sys.stderr, flush=True)

@@ -95,6 +95,23 @@ def gated_linear_large(x: torch.Tensor, w_gate_up: torch.Tensor):
 QKV_EPILOGUE = os.environ.get("DIB200_QKV_EPILOGUE", "1") != "0"
 
 
+def squared_relu_large(x: torch.Tensor, weight: torch.Tensor):
+    """max(x @ weight^T, 0)^2 for more than MAX_ROWS rows, the square in the tcgen05 product's epilogue, or
+    None if the shape does not allow it."""
+    from . import ops
+    m, k = x.shape
+    n = weight.shape[0]
+    if m <= MAX_ROWS or LARGE_PRODUCTS not in ("own", "auto") or k % 8 or n % 8 or weight.dtype != torch.bfloat16 \
+            or weight.shape[1] != k or x.data_ptr() % 16 or weight.data_ptr() % 16 or not x.is_contiguous() \
+            or not weight.is_contiguous():
+        return None
+    out = torch.empty(m, n, dtype=torch.bfloat16, device=x.device)
+    st = ops._lib("gemm_bf16_large").dib_gemm_bf16_large_squared_relu(
+        ops._ptr(x), ops._ptr(weight), ops._ptr(out), c_int(m), c_int(n), c_int(k), c_int(_sms(x.device)), ops._stream())
+    ops._check(st, "squared_relu_linear(bfloat16)", f"M={m} N={n} K={k}")
+    return out
+
+
 def qkv_large(x: torch.Tensor, w_qkv: torch.Tensor, num_heads: int, num_kv_heads: int, q_norm_weight,
               k_norm_weight, eps: float, cos_sin, positions, kv_cache, slot_mapping, page_size: int):
     """q [M, Hq, 128] of the fused projection with q/k norm, rotation and cache write in the

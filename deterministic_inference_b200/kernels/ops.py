@@ -628,7 +628,7 @@ def gather_rows(x: torch.Tensor, index: torch.Tensor) -> torch.Tensor:
     """out[r] = x[index[r]]; index int32."""
     if isinstance(x, NormedTerm):          # a norm works row by row: gather first
         return NormedTerm(gather_rows(x.x, index), x.weight, x.eps)
-    if isinstance(x, WeightedSum) and x.normed:
+    if isinstance(x, WeightedSum):
         return WeightedSum([(a, gather_rows(term, index)) for a, term in x.terms])
     x = as_tensor(x)
     _need(x, "x", None, 2)
@@ -899,6 +899,28 @@ def xielu(z, alpha_p: float, alpha_n: float, out_dtype) -> torch.Tensor:
                                       c_int(_DT[out_dtype]), c_longlong(rows * w), _stream())
     _check(st, "xielu")
     return out
+
+
+def squared_relu(z, out_dtype) -> torch.Tensor:
+    """max(z, 0)^2 in ``out_dtype``; float32 arithmetic."""
+    rows, w = z.shape
+    out = torch.empty(rows, w, dtype=out_dtype, device=z.device)
+    st = _lib("stream_f32").dib_squared_relu(*_source_args(z), _ptr(out), c_int(_DT[out_dtype]), c_longlong(rows * w),
+                                             _stream())
+    _check(st, "squared_relu")
+    return out
+
+
+def squared_relu_linear(x: torch.Tensor, weight: torch.Tensor, out_dtype) -> torch.Tensor:
+    """max(x @ weight^T, 0)^2, the square taken of the product's float32 sums.  Many bfloat16 rows: in the
+    product's epilogue; otherwise by a kernel that adds split-k partial products while it loads them."""
+    if x.dtype == torch.bfloat16 and out_dtype == torch.bfloat16:
+        from . import gemm_bf16
+        out = gemm_bf16.squared_relu_large(x, weight)
+        if out is not None:
+            return out
+    z = linear(x, weight, out_dtype=torch.float32 if x.dtype != torch.float32 else None)
+    return squared_relu(z, out_dtype)
 
 
 def scale_(x: torch.Tensor, a: float) -> torch.Tensor:
@@ -1223,6 +1245,75 @@ def state_space(proj, conv_weight: torch.Tensor, conv_bias, a_log: torch.Tensor,
     return out
 
 
+# ---------------------------------------------------------------- retention, a fixed decay per head
+
+# DIB200_RETENTION_CHUNKED=0 (read once): prompt portions run token by token too
+RETENTION_CHUNKED = __import__("os").environ.get("DIB200_RETENTION_CHUNKED", "1") != "0"
+
+
+def retention(proj, decay: torch.Tensor, freq, state: torch.Tensor, step, num_heads: int, head_dim: int,
+              v_head_dim: int, norm_eps: float, out_dtype) -> torch.Tensor:
+    """Retention over every sequence's tokens of the step: [T, H * E] in ``out_dtype``.  ``proj`` rows are
+    [q: H D | k: H D | v: H E | g: H E]; the first 2 * len(``freq``) elements of every q and k head turn in
+    halves (angle = position * freq; None: no rotation), k times D^(-1/2) behind it; per head S <-
+    decay[h] S + k v^T, o = S^T q, from and to ``state`` float32 [slots, H D E] (rows ``step.state_slots``);
+    then each head's o over its root mean square (``norm_eps``), times silu(g).  The step's leading
+    one-token sequences, and every sequence of the float32 engine or of sizes the chunked form does not
+    take, run token by token; other portions in chunks on the tensor cores, so which form a sequence
+    runs on depends on what IT brings."""
+    t, width = proj.shape
+    h, d, e = num_heads, head_dim, v_head_dim
+    if width < 2 * h * (d + e):
+        raise KernelError(f"retention: projection rows of {width}, expected at least {2 * h * (d + e)}")
+    _need(decay, "decay", torch.float32, 1)
+    _need(state, "state", torch.float32, 2)
+    if decay.shape[0] != h or state.shape[1] != h * d * e:
+        raise KernelError(f"retention: {decay.shape[0]} decays and state rows of {state.shape[1]} for {h} heads of {d}/{e}")
+    rot = 0
+    if freq is not None:
+        _need(freq, "freq", torch.float32, 1)
+        rot = 2 * freq.shape[0]
+        if rot > d:
+            raise KernelError(f"retention: a rotation of {rot} elements in heads of {d}")
+    lib = _lib("retention")
+    dev = state.device
+    out = torch.empty(t, h * e, dtype=out_dtype, device=dev)
+    n, nd = step.num_seqs, min(int(step.num_decode or 0), step.num_seqs)
+    chunked = RETENTION_CHUNKED and out_dtype == torch.bfloat16 and d % 16 == 0 and e % 16 == 0 and d <= 256 and e <= 256
+    if chunked and nd < n:
+        # (the step's own or padded projection rows as a stored bfloat16 matrix)
+        proj = as_tensor(proj)
+        chunked = proj.dtype == torch.bfloat16 and width % 8 == 0
+    k_scale = float(d) ** -0.5
+    stride = c_longlong(state.shape[1])
+
+    def by_token(first, count, in_smem):
+        st = lib.dib_retention_step(*_source_args(proj), c_longlong(width), _ptr(decay), _ptr(freq), c_int(rot),
+                                    _ptr(step.positions), _ptr(state), stride,
+                                    c_void_p(step.cu_q_lens.data_ptr() + 4 * first),
+                                    c_void_p(step.state_slots.data_ptr() + 4 * first), _ptr(out), c_int(_DT[out_dtype]),
+                                    c_int(count), c_int(h), c_int(d), c_int(e), c_float(k_scale), c_float(norm_eps),
+                                    c_int(in_smem), _stream())
+        _check(st, "retention(token by token)", f"heads of {d}/{e}")
+
+    if nd:
+        by_token(0, nd, 0)
+    if nd < n and not chunked:
+        by_token(nd, n - nd, int(lib.dib_retention_state_fits(c_int(d), c_int(e))))
+    elif nd < n:
+        tokens = t - nd
+        planes = torch.empty(4, tokens, h * d, dtype=torch.bfloat16, device=dev)
+        chunks = torch.empty(tokens // 64 + n - nd, h, d, e, dtype=torch.float32, device=dev)
+        st = lib.dib_retention_chunked(_ptr(proj), c_longlong(width), _ptr(decay), _ptr(freq), c_int(rot),
+                                       _ptr(step.positions), _ptr(state), stride,
+                                       c_void_p(step.cu_q_lens.data_ptr() + 4 * nd),
+                                       c_void_p(step.state_slots.data_ptr() + 4 * nd), _ptr(planes), _ptr(chunks),
+                                       _ptr(out), c_int(n - nd), c_int(nd), c_int(tokens), c_int(h), c_int(d), c_int(e),
+                                       c_float(k_scale), c_float(norm_eps), _stream())
+        _check(st, "retention(chunks)", f"heads of {d}/{e}", kernels=4)
+    return out
+
+
 # ---------------------------------------------------------------- gated linear recurrent unit
 
 def gated_linear_recurrence(proj, bias: torch.Tensor, conv_weight: torch.Tensor, conv_bias: torch.Tensor,
@@ -1315,26 +1406,48 @@ def route_experts(logits, correction: torch.Tensor, num_experts: int, top: int, 
     return ids, weights
 
 
-def routed_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
-                   w_down: torch.Tensor, shared, logits, shared_gate_col: int, out_dtype) -> torch.Tensor:
-    """float32 [T, W]: sum_j weights[t, j] * down_e(silu(gate_e x_t) * up_e x_t) over the chosen experts
-    e = ids[t, j], in the order of j, plus (``shared`` [T, W], a tensor or split sums, given)
+class TableChoice:
+    """A choice of experts that a table makes: token t's experts are the row ``table[token_ids[t]]``
+    (int32 [vocabulary, top]), each with the same ``weight``."""
+
+    def __init__(self, token_ids: torch.Tensor, table: torch.Tensor, weight: float):
+        self.token_ids, self.table, self.weight = token_ids, table, float(weight)
+
+
+def routed_experts(x: torch.Tensor, ids, weights, w_gate_up: torch.Tensor,
+                   w_down: torch.Tensor, shared, logits, shared_gate_col: int, out_dtype, limited=None) -> torch.Tensor:
+    """float32 [T, W]: sum_j weights[t, j] * down_e(act(gate_e x_t, up_e x_t)) over the chosen experts
+    e = ids[t, j], in the order of j (``ids`` a ``TableChoice``: the experts its table names, all with its
+    weight; ``weights`` None).  act(g, u) = silu(g) u, or with ``limited`` = (limit, alpha) min(g, limit)
+    sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1).  Plus (``shared`` [T, W], a tensor or split sums, given)
     sigmoid(logits[t, shared_gate_col]) * shared[t] (``shared_gate_col`` negative: plus shared[t]).  ``w_gate_up`` [E, 2F, W] (an expert's gate rows,
     then its up rows), ``w_down`` [E, W, F], both of x's type.  The (token, expert) pairs are sorted by
     expert on the device into tiles of EXPERT_TILE_ROWS (or EXPERT_TILE_ROWS_LARGE) rows of one expert; a
     row's sums run over k in an order that its tile does not change, so a token's result does not depend
     on what else is in the step."""
     _need(x, "x", None, 2)
-    _need(ids, "ids", torch.int32, 2)
-    _need(weights, "weights", torch.float32, 2)
+    table, weight = None, 0.0
+    if isinstance(ids, TableChoice):
+        if weights is not None:
+            raise KernelError("routed_experts: a table's choice brings its weight")
+        table, weight, ids = ids.table, ids.weight, ids.token_ids
+        _need(table, "table", torch.int32, 2)
+        _need(ids, "token ids", torch.int32, 1)
+        top = table.shape[1]
+    else:
+        _need(ids, "ids", torch.int32, 2)
+        _need(weights, "weights", torch.float32, 2)
+        top = ids.shape[1]
+    limit, alpha = (0.0, 0.0) if limited is None else (float(limited[0]), float(limited[1]))
+    if limited is not None and not limit > 0.0:
+        raise KernelError("routed_experts: the gate's limit is positive")
     _need(w_gate_up, "w_gate_up", x.dtype, 3)
     _need(w_down, "w_down", x.dtype, 3)
     t, w = x.shape
     n_exp, two_f, w2 = w_gate_up.shape
     f = two_f // 2
-    top = ids.shape[1]
-    if w2 != w or tuple(w_down.shape) != (n_exp, w, f) or two_f != 2 * f or tuple(weights.shape) != (t, top) \
-            or ids.shape[0] != t:
+    if w2 != w or tuple(w_down.shape) != (n_exp, w, f) or two_f != 2 * f or ids.shape[0] != t \
+            or (weights is not None and tuple(weights.shape) != (t, top)):
         raise KernelError(f"routed_experts: x {tuple(x.shape)}, gate/up {tuple(w_gate_up.shape)}, down "
                           f"{tuple(w_down.shape)}, ids {tuple(ids.shape)}")
     lib = _lib("routed_experts")
@@ -1346,7 +1459,7 @@ def routed_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_
         else EXPERT_TILE_ROWS_LARGE if pairs >= EXPERT_TILE_ROWS_LARGE * n_exp else EXPERT_TILE_ROWS
     max_tiles = pairs // tile + min(n_exp, pairs) + 1
     order = torch.empty(max_tiles * tile + max_tiles + n_exp + 2, dtype=torch.int32, device=dev)
-    st = lib.dib_moe_sort(_ptr(ids), c_int(pairs), c_int(n_exp), c_int(tile), c_int(max_tiles), _ptr(order), _stream())
+    st = lib.dib_moe_sort(_ptr(ids), _ptr(table), c_int(top), c_int(0 if table is None else table.shape[0]), c_int(pairs), c_int(n_exp), c_int(tile), c_int(max_tiles), _ptr(order), _stream())
     _check(st, "routed_experts(sort)", f"{n_exp} experts (at most 1024)")
     per_pair = torch.empty(pairs, w, dtype=torch.float32, device=dev)
     if on_tc:
@@ -1361,34 +1474,39 @@ def routed_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_
         hidden = torch.empty(rows, f, dtype=x.dtype, device=dev)
         st = large.dib_gemm_bf16_large_grouped(_ptr(sorted_x), _ptr(w_gate_up), _ptr(hidden), c_int(rows), c_int(f),
                                                c_int(w), c_int(1), c_int(0), tile_expert, c_int(n_exp),
-                                               c_int(_sms(dev)), _stream())
+                                               c_float(limit), c_float(alpha), c_int(_sms(dev)), _stream())
         _check(st, "routed_experts(gate and up, tcgen05)", f"rows {rows}, F {f}, W {w}")
         sorted_y = torch.empty(rows, w, dtype=torch.float32, device=dev)
         st = large.dib_gemm_bf16_large_grouped(_ptr(hidden), _ptr(w_down), _ptr(sorted_y), c_int(rows), c_int(w),
                                                c_int(f), c_int(0), c_int(1), tile_expert, c_int(n_exp),
-                                               c_int(_sms(dev)), _stream())
+                                               c_float(0.0), c_float(0.0), c_int(_sms(dev)), _stream())
         _check(st, "routed_experts(down, tcgen05)", f"rows {rows}, F {f}, W {w}")
         st = lib.dib_moe_scatter_rows(_ptr(sorted_y), _ptr(order), c_longlong(rows), c_int(w), _ptr(per_pair), _stream())
         _check(st, "routed_experts(rows back to their pairs)")
     else:
         hidden = torch.empty(max_tiles * tile, f, dtype=x.dtype, device=dev)
         st = lib.dib_moe_gate_up(_ptr(x), c_int(_dt(x, "x")), _ptr(order), c_int(max_tiles), c_int(tile), c_int(top),
-                                 _ptr(w_gate_up), _ptr(hidden), c_int(f), c_int(w), _stream())
+                                 _ptr(w_gate_up), _ptr(hidden), c_int(f), c_int(w), c_float(limit), c_float(alpha),
+                                 _stream())
         _check(st, "routed_experts(gate and up)")
         st = lib.dib_moe_down(_ptr(hidden), c_int(_dt(x, "x")), _ptr(order), c_int(max_tiles), c_int(tile), _ptr(w_down),
                               _ptr(per_pair), c_int(f), c_int(w), _stream())
         _check(st, "routed_experts(down)")
     out = torch.empty(t, w, dtype=torch.float32, device=dev)
     if shared is not None:
-        if tuple(shared.shape) != (t, w) or logits.shape[0] != t or logits.shape[1] <= shared_gate_col:
-            raise KernelError(f"routed_experts: shared output {tuple(shared.shape)}, logits {tuple(logits.shape)}")
-        sh, lg, row = _source_args(shared), _source_args(logits), logits.shape[1]
+        if tuple(shared.shape) != (t, w) or (shared_gate_col >= 0 and (
+                logits is None or logits.shape[0] != t or logits.shape[1] <= shared_gate_col)):
+            raise KernelError(f"routed_experts: shared output {tuple(shared.shape)} for {(t, w)}, or logits that do not "
+                              f"hold its gate in column {shared_gate_col}")
+        sh = _source_args(shared)
         if shared_gate_col < 0:
-            shared_gate_col = -1
+            shared_gate_col, lg, row = -1, (c_void_p(0), c_int(0), c_int(1), c_longlong(0)), 0
+        else:
+            lg, row = _source_args(logits), logits.shape[1]
     else:
         sh = lg = (c_void_p(0), c_int(0), c_int(1), c_longlong(0))
         row = 0
-    st = lib.dib_moe_combine(_ptr(per_pair), _ptr(weights), *sh, *lg, c_longlong(row), c_int(shared_gate_col),
+    st = lib.dib_moe_combine(_ptr(per_pair), _ptr(weights), c_float(weight), *sh, *lg, c_longlong(row), c_int(shared_gate_col),
                              _ptr(out), c_int(t), c_int(top), c_int(w), _stream())
     _check(st, "routed_experts(combine)")
     return out
@@ -1508,19 +1626,27 @@ def attn_prepare(proj, num_heads: int, num_kv_heads: int, head_dim: int, v_head_
 
 
 def latent_prepare(proj, num_heads: int, plain_dim: int, rot_dim: int, rank: int, latent_norm_weight,
-                   eps: float, freq, positions, kv_cache, slot_mapping, page_size: int, out_dtype) -> torch.Tensor:
+                   eps: float, freq, positions, kv_cache, slot_mapping, page_size: int, out_dtype,
+                   rotary_layout: str = "halves", amplitude: float = 1.0) -> torch.Tensor:
     """From each token's projection row [q: heads of (plain_dim + rot_dim) | latent: rank | rotated key
     part: rot_dim]: the latent, RMS-normed with its weight, and the rotated key part go to the token's
     cache row [rank + rot_dim]; the rotated part of every query head goes to q[t, h, rank:], where q
     [T, H, rank + rot_dim] is returned with its first ``rank`` columns still to be filled (by the
-    product of the head's plain part with its key map)."""
+    product of the head's plain part with its key map).  ``rotary_layout`` "halves": element i of a
+    rotated part turns with i + rot_dim / 2, "pairs": 2i with 2i + 1; cosine and sine times ``amplitude``.
+    ``latent_norm_weight`` None: a layer that reads another layer's cached rows; its projection row is
+    the query heads alone and nothing is stored."""
     t, width = proj.shape
-    if width != num_heads * (plain_dim + rot_dim) + rank + rot_dim:
+    own = latent_norm_weight is not None
+    if width != num_heads * (plain_dim + rot_dim) + (rank + rot_dim if own else 0):
         raise KernelError(f"latent_prepare: rows of {width} elements, expected "
-                          f"{num_heads * (plain_dim + rot_dim) + rank + rot_dim}")
-    _need(latent_norm_weight, "latent_norm_weight", torch.float32, 1)
+                          f"{num_heads * (plain_dim + rot_dim) + (rank + rot_dim if own else 0)}")
+    if rotary_layout not in ("halves", "pairs") or (not own and kv_cache is not None):
+        raise KernelError(f"latent_prepare: rotary layout {rotary_layout!r}, or a cache to write without a latent")
+    if own:
+        _need(latent_norm_weight, "latent_norm_weight", torch.float32, 1)
     _need(freq, "freq", torch.float32, 1)
-    if freq.shape[0] * 2 != rot_dim or latent_norm_weight.shape[0] != rank:
+    if freq.shape[0] * 2 != rot_dim or (own and latent_norm_weight.shape[0] != rank):
         raise KernelError("latent_prepare: frequencies or norm weight of the wrong size")
     _need(positions, "positions", torch.int32, 1)
     num_pages = 0
@@ -1532,7 +1658,8 @@ def latent_prepare(proj, num_heads: int, plain_dim: int, rot_dim: int, rank: int
     st = _lib("masked_attention").dib_latent_prepare(
         *_source_args(proj), c_longlong(width), _ptr(q), _ptr(kv_cache), _ptr(latent_norm_weight), c_float(eps),
         _ptr(freq), _ptr(positions), _ptr(slot_mapping), c_int(t), c_int(num_heads), c_int(plain_dim),
-        c_int(rot_dim), c_int(rank), c_int(page_size), c_longlong(num_pages), c_int(_DT[out_dtype]), _stream())
+        c_int(rot_dim), c_int(rank), c_int(page_size), c_longlong(num_pages), c_int(_DT[out_dtype]),
+        c_int(1 if rotary_layout == "pairs" else 0), c_float(amplitude), _stream())
     _check(st, "latent_prepare")
     return q
 

@@ -19,6 +19,7 @@ from ..config.bovitar_config import BovitarConfig
 from ..config.gamilorn_config import GamilornConfig
 from ..config.kipezen_config import KipezenConfig
 from ..config.model_config import Qwen3Config
+from ..config.nedupel_config import NedupelConfig
 from ..config.zatirax_config import ZatiraxConfig
 from .decoder import DecoderModel
 
@@ -39,6 +40,7 @@ register_architecture("Gamilorn", GamilornConfig)
 register_architecture("Zatirax", ZatiraxConfig)
 register_architecture("Kipezen", KipezenConfig)
 register_architecture("Bovitar", BovitarConfig)
+register_architecture("Nedupel", NedupelConfig)
 
 
 def config_from_dir(model_dir):

@@ -8,7 +8,8 @@ Norm(Part)           forward(x) -> y;  add_forward(x, residual) -> (y, residual)
 PositionEncoding     prepare(); rotary_table() -> Tensor | None; apply(q, k, positions)
 Mixer(Part)          cache_spec() -> PagedKVSpec | StateSpec | None
                      forward(x [T, H], step, cache) -> [T, H]
-FeedForward(Part)    forward(x [T, H]) -> [T, H]
+FeedForward(Part)    forward(x [T, H]) -> [T, H];  ``needs_step``: forward(x, step) (it reads the
+                     step's token ids)
 Block                forward(hidden, residual, step, cache) -> (hidden, residual)
 
 What a mixer or feed-forward returns, and what a block hands on as ``hidden``, is a
@@ -87,6 +88,11 @@ class Mixer(Part):
 
 
 class FeedForward(Part):
+    needs_step = False
+
+    def run(self, x: torch.Tensor, step) -> torch.Tensor:
+        return self.forward(x, step) if self.needs_step else self.forward(x)
+
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
 

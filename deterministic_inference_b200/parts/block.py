@@ -28,7 +28,7 @@ class PreNormBlock(Block):
             hidden, residual = self.mixer_norm.add_forward(hidden, residual)
         hidden = self.mixer.forward(hidden, step, cache)
         hidden, residual = self.feed_forward_norm.add_forward(hidden, residual)
-        hidden = self.feed_forward.forward(hidden)
+        hidden = self.feed_forward.run(hidden, step)
         return hidden, residual
 
 
@@ -38,11 +38,19 @@ class PreNormStreamBlock(Block):
     x <- x + feed_forward(norm(x)), every addition in float32 whatever type the parts
     compute in.  The stream comes in as float32 (from the embedding, or as the stream and
     the pending output of the layer before); a layer without a feed-forward (kind "none")
-    hands its mixer's output on as the pending term."""
+    hands its mixer's output on as the pending term.  ``branch_scale`` m: x <- x + m * mixer(norm(x))
+    and so on; the factor is applied where the pending term joins the stream (``ops.WeightedSum``)."""
 
-    def __init__(self, ctx, mixer, feed_forward, mixer_norm, feed_forward_norm):
+    def __init__(self, ctx, mixer, feed_forward, mixer_norm, feed_forward_norm, branch_scale: float = 1.0):
         self.mixer, self.feed_forward = mixer, feed_forward
         self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
+        self.branch_scale = float(branch_scale)
+
+    def _scaled(self, out):
+        if self.branch_scale == 1.0:
+            return out
+        terms = out.terms if isinstance(out, ops.WeightedSum) else [(1.0, out)]
+        return ops.WeightedSum([(self.branch_scale * a, x) for a, x in terms])
 
     def forward(self, hidden, residual, step, cache):
         if residual is None:
@@ -50,11 +58,11 @@ class PreNormStreamBlock(Block):
             hidden = self.mixer_norm.forward(residual)
         else:
             hidden, residual = self.mixer_norm.add_forward(hidden, residual)
-        hidden = self.mixer.forward(hidden, step, cache)
+        hidden = self._scaled(self.mixer.forward(hidden, step, cache))
         if self.feed_forward.kind == "none":
             return hidden, residual
         hidden, residual = self.feed_forward_norm.add_forward(hidden, residual)
-        hidden = self.feed_forward.forward(hidden)
+        hidden = self._scaled(self.feed_forward.run(hidden, step))
         return hidden, residual
 
 
@@ -86,7 +94,7 @@ class SandwichStreamBlock(Block):
         if self.feed_forward.kind == "none":
             return hidden, residual
         hidden, residual = self.feed_forward_norm.add_forward(hidden, residual)
-        hidden = self.feed_forward_post_norm.forward(self.feed_forward.forward(hidden))
+        hidden = self.feed_forward_post_norm.forward(self.feed_forward.run(hidden, step))
         return hidden, residual
 
 
@@ -112,5 +120,5 @@ class PostNormStreamBlock(Block):
         if self.feed_forward.kind == "none":
             return hidden, residual
         x = ops.stream_read(residual, hidden, self.dtype)
-        hidden = self.feed_forward_norm.forward(self.feed_forward.forward(x))
+        hidden = self.feed_forward_norm.forward(self.feed_forward.run(x, step))
         return hidden, residual

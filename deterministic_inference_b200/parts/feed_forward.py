@@ -52,7 +52,8 @@ class GatedMLP(FeedForward):
 
 @register_feed_forward("dense_mlp")
 class DenseMLP(FeedForward):
-    """down( act(up(x)) ), no gate and no biases.  ``activation`` "xielu": with the two stored
+    """down( act(up(x)) ), no gate and no biases.  ``activation`` "squared_relu": max(z, 0)^2, in
+    float32 from the product's accumulator where it is at hand.  "xielu": with the two stored
     numbers p, q of ``act_name`` and softplus(y) = log(1 + exp(y)),
     act(z) = softplus(p) z^2 + z / 2 for z > 0 and (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2
     otherwise, computed in float32 from the product's accumulator where it is at hand."""
@@ -60,9 +61,9 @@ class DenseMLP(FeedForward):
     def __init__(self, ctx, prefix: str, hidden_size: int, intermediate_size: int,
                  activation: str = "xielu", up_name: str = "up", down_name: str = "down",
                  act_name: str = "act"):
-        if activation != "xielu":
-            raise ValueError(f"dense_mlp: activation {activation!r} has no kernel (only 'xielu')")
-        self.prefix, self.names = prefix, (up_name, down_name, act_name)
+        if activation not in ("xielu", "squared_relu"):
+            raise ValueError(f"dense_mlp: activation {activation!r} has no kernel ('xielu', 'squared_relu')")
+        self.prefix, self.activation, self.names = prefix, activation, (up_name, down_name, act_name)
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.out_dtype = ctx.dtype
         self.w_up = self.w_down = None
@@ -71,16 +72,22 @@ class DenseMLP(FeedForward):
     def tensor_specs(self):
         p, h, i = self.prefix, self.hidden_size, self.intermediate_size
         up, down, act = self.names
-        return [TensorSpec(p + up, (i, h)), TensorSpec(p + down, (h, i)),
-                TensorSpec(p + act, (2,), role="vector")]
+        specs = [TensorSpec(p + up, (i, h)), TensorSpec(p + down, (h, i))]
+        if self.activation == "xielu":
+            specs.append(TensorSpec(p + act, (2,), role="vector"))
+        return specs
 
     def load(self, tensors):
         up, down, act = self.names
         self.w_up, self.w_down = tensors[self.prefix + up], tensors[self.prefix + down]
+        if self.activation != "xielu":
+            return
         pq = torch.nn.functional.softplus(tensors[self.prefix + act].to("cpu", torch.float32))
         self.alpha_p, self.alpha_n = float(pq[0]), float(torch.tensor(0.5, dtype=torch.float32) + pq[1])
 
     def forward(self, x):
+        if self.activation == "squared_relu":
+            return ops.linear(ops.squared_relu_linear(x, self.w_up, self.out_dtype), self.w_down)
         z = ops.linear(x, self.w_up, out_dtype=torch.float32 if x.dtype != torch.float32 else None)
         return ops.linear(ops.xielu(z, self.alpha_p, self.alpha_n, self.out_dtype), self.w_down)
 

@@ -15,7 +15,11 @@ the cached rows [c | k_r] as ONE key head of kv_rank + rot_dim elements whose fi
 elements double as the value, and the weighted latent goes through the value map.  A token costs
 kv_rank + rot_dim cache elements whatever the number of heads.  Softmax over the keys the mask
 shows ("causal", "window", "chunk" as in ``masked_attention``); norms, angles, scores and the softmax
-are float32.
+are float32.  ``rotary_layout``: "halves" (element i of a rotated part turns with i + rot_dim / 2) or
+"pairs" (2i with 2i + 1); the position encoding's ``amplitude`` multiplies cosine and sine.
+
+``own_latent`` off: the layer has no W_dkv and reads the rows that another layer of the same
+kv_rank, rot_dim and rotation left in the cache its schedule entry names.
 """
 
 from __future__ import annotations
@@ -34,12 +38,16 @@ from .spec import PagedKVSpec, PartSpec, TensorSpec
 class LatentAttention(Mixer):
     def __init__(self, ctx, prefix: str, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int,
                  v_head_dim: int, kv_rank: int, scale: float, position_encoding: PartSpec, norm_eps: float,
-                 mask: str = "causal", mask_size: Optional[int] = None, names: Optional[dict] = None):
+                 mask: str = "causal", mask_size: Optional[int] = None, names: Optional[dict] = None,
+                 rotary_layout: str = "halves", own_latent: bool = True):
         if mask not in ("causal", "window", "chunk"):
             raise ValueError(f"mask {mask!r} is not known ('causal', 'window', 'chunk')")
         if mask != "causal" and (mask_size is None or int(mask_size) < 1):
             raise ValueError(f"a {mask} mask needs a positive mask_size")
+        if rotary_layout not in ("halves", "pairs"):
+            raise ValueError(f"rotary_layout {rotary_layout!r} is not known ('halves', 'pairs')")
         self.prefix = prefix
+        self.rotary_layout, self.own_latent = rotary_layout, bool(own_latent)
         self.hidden_size, self.num_heads = int(hidden_size), int(num_heads)
         self.head_dim, self.rot_dim, self.v_head_dim = int(head_dim), int(rot_dim), int(v_head_dim)
         self.kv_rank, self.scale, self.norm_eps = int(kv_rank), float(scale), float(norm_eps)
@@ -56,16 +64,21 @@ class LatentAttention(Mixer):
     def tensor_specs(self):
         p, n, w = self.prefix, self.names, self.hidden_size
         h, d, r, e, c = self.num_heads, self.head_dim, self.rot_dim, self.v_head_dim, self.kv_rank
-        return [TensorSpec(p + n["q"], (h * (d + r), w)), TensorSpec(p + n["down"], (c + r, w)),
-                TensorSpec(p + n["latent_norm"], (c,), role="vector", init="one_plus_normal"),
-                TensorSpec(p + n["key_map"], (h * d, c)), TensorSpec(p + n["value_map"], (h * e, c)),
-                TensorSpec(p + n["o"], (w, h * e))]
+        specs = [TensorSpec(p + n["q"], (h * (d + r), w))]
+        if self.own_latent:
+            specs += [TensorSpec(p + n["down"], (c + r, w)),
+                      TensorSpec(p + n["latent_norm"], (c,), role="vector", init="one_plus_normal")]
+        return specs + [TensorSpec(p + n["key_map"], (h * d, c)), TensorSpec(p + n["value_map"], (h * e, c)),
+                        TensorSpec(p + n["o"], (w, h * e))]
 
     def load(self, tensors):
         p, n = self.prefix, self.names
         h, d, e, c = self.num_heads, self.head_dim, self.v_head_dim, self.kv_rank
-        self.w_in = torch.cat([tensors[p + n["q"]], tensors[p + n["down"]]], dim=0).contiguous()
-        self.latent_norm = tensors[p + n["latent_norm"]]
+        if self.own_latent:
+            self.w_in = torch.cat([tensors[p + n["q"]], tensors[p + n["down"]]], dim=0).contiguous()
+            self.latent_norm = tensors[p + n["latent_norm"]]
+        else:
+            self.w_in = tensors[p + n["q"]]
         # per head [K, N]: the key map takes a query's plain part [d] to the latent's size [c]; the
         # value map takes a weighted latent [c] to the head's value [e]
         self.w_key = tensors[p + n["key_map"]].view(h, d, c).contiguous()
@@ -82,8 +95,9 @@ class LatentAttention(Mixer):
         proj = ops.as_tensor(ops.linear(x, self.w_in))
         t, width = proj.shape
         q = ops.latent_prepare(proj, h, d, r, c, self.latent_norm, self.norm_eps, self.freq, step.positions,
-                               cache.kv if cache.writes else None, cache.slot_mapping, cache.page_size,
-                               self.out_dtype)
+                               cache.kv if cache.writes and self.own_latent else None, cache.slot_mapping,
+                               cache.page_size, self.out_dtype, rotary_layout=self.rotary_layout,
+                               amplitude=self.position_encoding.amplitude)
         ops.heads_linear(proj.as_strided((t, h, d), (width, d + r, 1)), self.w_key, q[:, :, :c])
         latent = ops.masked_attention(q, cache.kv, cache.attention_meta, self.scale, 1, c, cache.page_size,
                                       self.mask, self.mask_size, values_in_keys=True)

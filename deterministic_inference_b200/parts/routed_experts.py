@@ -1,7 +1,10 @@
 """A feed-forward of routed experts beside a shared expert.
 
-``num_experts`` gated feed-forwards (W_down (silu(W_gate x) * (W_up x)), no biases), of which each
-token uses ``top``.  Router: z = W_router x in float32, scores s = sigmoid(z) or (``score``
+``num_experts`` gated feed-forwards (W_down act(W_gate x, W_up x), no biases), of which each
+token uses ``top``.  ``activation`` "silu": silu(g) u; "limited_swish": with g = min(g, limit) and u =
+clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1).  ``score`` "table": no router; a stored table
+[vocabulary, top] of integers gives each token id its experts, each with weight ``route_scale`` / top.
+Otherwise, router: z = W_router x in float32, scores s = sigmoid(z) or (``score``
 "softmax") softmax(z) over all experts.  The choice is made on s + correction (a stored vector),
 the weights use s without it.  The experts form ``group_count`` equal groups of neighbours; a
 group's score is the sum of its ``group_top`` largest choice scores (2, or 1: its largest), and only
@@ -30,10 +33,19 @@ class RoutedExperts(FeedForward):
                  route_scale: float, group_count: int = 1, group_keep: int = 1,
                  shared_intermediate_size: Optional[int] = None, weight_eps: float = 1e-20,
                  names: Optional[dict] = None, score: str = "sigmoid", group_top: int = 2, normalize: bool = True,
-                 shared_gate: bool = True):
-        if score not in ops.ROUTER_SCORES or int(group_top) not in (1, 2):
-            raise ValueError(f"routed_experts: score {score!r} ({sorted(ops.ROUTER_SCORES)}) or group_top "
+                 shared_gate: bool = True, activation: str = "silu", limit: Optional[float] = None,
+                 alpha: float = 1.702, vocab_size: Optional[int] = None):
+        if (score != "table" and score not in ops.ROUTER_SCORES) or int(group_top) not in (1, 2):
+            raise ValueError(f"routed_experts: score {score!r} ({sorted(ops.ROUTER_SCORES)}, 'table') or group_top "
                              f"{group_top!r} (1, 2) is not known")
+        if activation not in ("silu", "limited_swish"):
+            raise ValueError(f"routed_experts: activation {activation!r} has no kernel ('silu', 'limited_swish')")
+        if activation == "limited_swish" and (limit is None or not float(limit) > 0):
+            raise ValueError("routed_experts: 'limited_swish' needs a positive limit")
+        if score == "table" and (vocab_size is None or shared_gate and shared_intermediate_size is not None
+                                 or group_count != 1):
+            raise ValueError("routed_experts: a table of choices needs vocab_size, and has no groups and no gate for "
+                             "a shared expert (their numbers come from a router)")
         if num_experts % group_count or group_keep > group_count or top > group_keep * (num_experts // group_count):
             raise ValueError(f"routed_experts: {num_experts} experts in {group_count} groups, {group_keep} kept, "
                              f"{top} chosen do not fit")
@@ -45,11 +57,14 @@ class RoutedExperts(FeedForward):
         self.shared_size = None if shared_intermediate_size is None else int(shared_intermediate_size)
         self.score, self.group_top, self.normalize = score, int(group_top), bool(normalize)
         self.shared_gate = bool(shared_gate) and self.shared_size is not None
+        self.limited = (float(limit), float(alpha)) if activation == "limited_swish" else None
+        self.vocab_size = None if vocab_size is None else int(vocab_size)
+        self.needs_step = score == "table"          # the choice is made on the step's token ids
         self.names = dict(expert="e{}.", gate="gate", up="up", down="down", router="router",
-                          correction="correction", shared="shared.", shared_gate="shared.sg")
+                          correction="correction", shared="shared.", shared_gate="shared.sg", table="table")
         self.names.update(names or {})
         self.out_dtype = ctx.dtype
-        self.w_router = self.correction = self.w_gate_up = self.w_down = None
+        self.w_router = self.correction = self.w_gate_up = self.w_down = self.table = None
         self.shared_gate_up = self.shared_down = None
 
     def tensor_specs(self):
@@ -59,8 +74,12 @@ class RoutedExperts(FeedForward):
             q = p + n["expert"].format(e)
             specs += [TensorSpec(q + n["gate"], (f, w)), TensorSpec(q + n["up"], (f, w)),
                       TensorSpec(q + n["down"], (w, f))]
-        specs += [TensorSpec(p + n["router"], (self.num_experts, w)),
-                  TensorSpec(p + n["correction"], (self.num_experts,), role="vector", init="normal")]
+        if self.score == "table":
+            specs.append(TensorSpec(p + n["table"], (self.vocab_size, self.top), role="index", init="distinct",
+                                    high=self.num_experts))
+        else:
+            specs += [TensorSpec(p + n["router"], (self.num_experts, w)),
+                      TensorSpec(p + n["correction"], (self.num_experts,), role="vector", init="normal")]
         if self.shared_size is not None:
             q, s = p + n["shared"], self.shared_size
             specs += [TensorSpec(q + n["gate"], (s, w)), TensorSpec(q + n["up"], (s, w)),
@@ -76,28 +95,41 @@ class RoutedExperts(FeedForward):
         self.w_gate_up = torch.stack([torch.cat([tensors[q + n["gate"]], tensors[q + n["up"]]], dim=0)
                                       for q in names]).contiguous()
         self.w_down = torch.stack([tensors[q + n["down"]] for q in names]).contiguous()
+        if self.shared_size is not None:
+            q = p + n["shared"]
+            self.shared_gate_up = torch.cat([tensors[q + n["gate"]], tensors[q + n["up"]]], dim=0).contiguous()
+            self.shared_down = tensors[q + n["down"]]
+        if self.score == "table":
+            self.table = tensors[p + n["table"]]
+            return
         # one product gives the router's logits and, behind them, the shared expert's gate; its rows are
         # filled up to a multiple of 8 with zeros
         rows = [tensors[p + n["router"]]]
-        if self.shared_size is not None:
-            q = p + n["shared"]
-            if self.shared_gate:
-                rows.append(tensors[p + n["shared_gate"]])
-            self.shared_gate_up = torch.cat([tensors[q + n["gate"]], tensors[q + n["up"]]], dim=0).contiguous()
-            self.shared_down = tensors[q + n["down"]]
+        if self.shared_gate:
+            rows.append(tensors[p + n["shared_gate"]])
         have = sum(r.shape[0] for r in rows)
         if have % 8:
             rows.append(torch.zeros(8 - have % 8, self.hidden_size, dtype=rows[0].dtype, device=rows[0].device))
         self.w_router = torch.cat(rows, dim=0).contiguous()
         self.correction = tensors[p + n["correction"]]
 
-    def forward(self, x):
+    def _shared(self, x):
+        if self.shared_size is None:
+            return None
+        if self.limited is not None:
+            gate_up = ops.linear(x, self.shared_gate_up)
+            return ops.linear(ops.limited_gate(gate_up, *self.limited, self.out_dtype), self.shared_down)
+        return ops.linear(ops.gated_linear(x, self.shared_gate_up), self.shared_down)
+
+    def forward(self, x, step=None):
+        if self.score == "table":
+            choice = ops.TableChoice(step.input_ids, self.table, self.route_scale / self.top)
+            return ops.routed_experts(x, choice, None, self.w_gate_up, self.w_down, self._shared(x), None, -1,
+                                      self.out_dtype, limited=self.limited)
         logits = ops.linear(x, self.w_router, out_dtype=torch.float32 if x.dtype != torch.float32 else None)
         ids, weights = ops.route_experts(logits, self.correction, self.num_experts, self.top, self.group_count,
                                          self.group_keep, self.route_scale, self.weight_eps, score=self.score,
                                          group_top=self.group_top, normalize=self.normalize)
-        shared = None
-        if self.shared_size is not None:
-            shared = ops.linear(ops.gated_linear(x, self.shared_gate_up), self.shared_down)
-        return ops.routed_experts(x, ids, weights, self.w_gate_up, self.w_down, shared, logits,
-                                  self.num_experts if self.shared_gate else -1, self.out_dtype)
+        return ops.routed_experts(x, ids, weights, self.w_gate_up, self.w_down, self._shared(x), logits,
+                                  self.num_experts if self.shared_gate else -1, self.out_dtype,
+                                  limited=self.limited)

@@ -95,13 +95,17 @@ class TensorSpec:
     role "table":  the embedding [vocab, hidden], cast to the engine dtype.
     role "vector": a norm weight; kept in float32 whatever it is stored as
                    (norm math is float32).
+    role "index":  a table of integers, stored as integers and kept as int32; the entries of a
+                   row are distinct and lie in [0, ``high``).
     ``init`` names the law the random-weights mode draws it from.
     """
 
     name: str
     shape: tuple
     role: str = "matrix"
-    init: str = "normal"          # "normal": N(0, std); "one_plus_normal": 1 + N(0, norm_std)
+    init: str = "normal"          # "normal": N(0, std); "one_plus_normal": 1 + N(0, norm_std);
+                                  # "distinct": every row distinct integers below ``high``
+    high: int = 0
 
 
 @dataclass(frozen=True)

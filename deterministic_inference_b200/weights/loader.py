@@ -10,7 +10,8 @@ everything that is missing, unexpected or of the wrong shape or type.
 dtype: matrices and the embedding are cast to the engine dtype (bfloat16, or
 float32 for the 32-bit path, which upcasts exactly); norm weights are kept in
 float32 whatever they are stored as, because norm arithmetic is float32; an
-integer tensor would be kept as int32.
+integer tensor (role "index") is kept as int32, with its entries checked against the
+range the part gives.
 """
 
 from __future__ import annotations
@@ -63,7 +64,10 @@ def check_checkpoint(headers: dict[str, dict], specs: list[TensorSpec], plan: Mo
         got = tuple(headers[n]["shape"])
         if got != tuple(s.shape):
             wrong_shape.append(f"{n}: expected {list(s.shape)}, found {list(got)}")
-        if headers[n]["dtype"] not in _FLOAT_CODES:
+        if s.role == "index":
+            if headers[n]["dtype"] not in _INT_CODES:
+                wrong_type.append(f"{n}: stored as {headers[n]['dtype']}, expected an integer type")
+        elif headers[n]["dtype"] not in _FLOAT_CODES:
             wrong_type.append(f"{n}: stored as {headers[n]['dtype']}, expected a floating type")
     if missing or unexpected or wrong_shape or wrong_type:
         lines = ["checkpoint does not match the model:"]
@@ -105,5 +109,8 @@ def load_weights(model_dir, specs: list[TensorSpec], plan: ModelPlan, dtype: tor
         with safe_open(str(f), framework="pt", device="cpu") as reader:
             for s in wanted:
                 t = reader.get_tensor(s.name)
+                if s.role == "index" and t.numel() and not (0 <= int(t.min()) and int(t.max()) < s.high):
+                    raise WeightsError(f"{s.name}: entries from {int(t.min())} to {int(t.max())}, "
+                                       f"expected integers in [0, {s.high})")
                 out[s.name] = t.to(device=device, dtype=target_dtype(s, t.dtype, dtype)).contiguous()
     return out

@@ -6,7 +6,7 @@ Law: matrices and the embedding N(0, std), norm weights 1 + N(0, norm_std), draw
 in float32 from ONE ``torch.Generator`` seeded once, in the fixed order in which
 the model lists its tensors, then stored as bfloat16 like a published
 checkpoint.  Both engine dtypes therefore run the same values (the 32-bit path
-upcasts them exactly).
+upcasts them exactly).  Integer tables: every row distinct integers of the table's range, int32.
 """
 
 from __future__ import annotations
@@ -19,11 +19,26 @@ import torch
 from ..parts.spec import TensorSpec
 
 
+def _distinct_rows(spec: TensorSpec, generator, device) -> torch.Tensor:
+    """int32 [rows, n]: the places of the n largest of ``high`` uniform numbers a row."""
+    rows, n = spec.shape
+    if n > spec.high:
+        raise ValueError(f"{spec.name}: rows of {n} distinct integers below {spec.high}")
+    out = torch.empty(rows, n, dtype=torch.int32, device=device)
+    for a in range(0, rows, 4096):
+        x = torch.rand(min(4096, rows - a), spec.high, generator=generator, device=device)
+        out[a:a + x.shape[0]] = x.topk(n, dim=-1).indices.to(torch.int32)
+    return out
+
+
 def random_tensors(specs: list[TensorSpec], seed: int, std: float = 0.02, norm_std: float = 0.1,
                    store_dtype: torch.dtype = torch.bfloat16) -> dict[str, torch.Tensor]:
     g = torch.Generator(device="cpu").manual_seed(int(seed))
     out = {}
     for s in specs:
+        if s.init == "distinct":
+            out[s.name] = _distinct_rows(s, g, "cpu")
+            continue
         x = torch.randn(tuple(s.shape), generator=g, dtype=torch.float32)
         if s.init == "one_plus_normal":
             x = 1.0 + norm_std * x
@@ -44,6 +59,9 @@ def random_tensors_on_device(specs: list[TensorSpec], seed: int, dtype: torch.dt
     out = {}
     for i, s in enumerate(specs):
         g = torch.Generator(device=device).manual_seed(int(seed) * 1_000_003 + i)
+        if s.init == "distinct":
+            out[s.name] = _distinct_rows(s, g, device)
+            continue
         x = torch.randn(tuple(s.shape), generator=g, dtype=torch.float32, device=device)
         if s.init == "one_plus_normal":
             x = 1.0 + norm_std * x

@@ -408,16 +408,17 @@ def attn_prepare(proj, num_heads, num_kv_heads, head_dim, v_head_dim, q_norm_wei
 
 
 def latent_prepare(proj, num_heads, plain_dim, rot_dim, rank, latent_norm_weight, eps, freq, positions, kv_cache,
-                   slot_mapping, page_size, out_dtype):
+                   slot_mapping, page_size, out_dtype, rotary_layout="halves", amplitude=1.0):
     x = _plain(proj).to(out_dtype).float()
     t = x.shape[0]
     nq = num_heads * (plain_dim + rot_dim)
+    turn = _rotate_pairs if rotary_layout == "pairs" else _rotate_first
     q_rot = x[:, :nq].reshape(t, num_heads, plain_dim + rot_dim)[:, :, plain_dim:]
     q = torch.zeros(t, num_heads, rank + rot_dim, dtype=out_dtype)
-    q[:, :, rank:] = _rotate_first(q_rot, positions, freq, rot_dim).to(out_dtype)
+    q[:, :, rank:] = (amplitude * turn(q_rot, positions, freq, rot_dim)).to(out_dtype)
     if kv_cache is not None:
         latent = _rms(x[:, nq:nq + rank], latent_norm_weight, eps)
-        k_rot = _rotate_first(x[:, None, nq + rank:], positions, freq, rot_dim)[:, 0]
+        k_rot = amplitude * turn(x[:, None, nq + rank:], positions, freq, rot_dim)[:, 0]
         rows = kv_cache.view(-1, rank + rot_dim)
         for i, slot in enumerate(slot_mapping.tolist()[:t]):
             if slot >= 0:
@@ -592,15 +593,54 @@ def route_experts(logits, correction, num_experts, top, group_count, group_keep,
     return ids.to(torch.int32), w
 
 
-def routed_experts(x, ids, weights, w_gate_up, w_down, shared, logits, shared_gate_col, out_dtype):
+def squared_relu(z, out_dtype):
+    return torch.relu(_plain(z)).square().to(out_dtype)
+
+
+def squared_relu_linear(x, weight, out_dtype):
+    return torch.relu(x.float() @ weight.float().T).square().to(out_dtype)
+
+
+def retention(proj, decay, freq, state, step, num_heads, head_dim, v_head_dim, norm_eps, out_dtype):
+    h, d, e = num_heads, head_dim, v_head_dim
+    x = _plain(proj).to(out_dtype).float()
+    t = x.shape[0]
+    q, k = x[:, :h * d].reshape(t, h, d), x[:, h * d:2 * h * d].reshape(t, h, d)
+    v, g = x[:, 2 * h * d:2 * h * d + h * e].reshape(t, h, e), x[:, 2 * h * d + h * e:2 * h * (d + e)]
+    if freq is not None:
+        q = _rotate_first(q, step.positions, freq, 2 * freq.shape[0])
+        k = _rotate_first(k, step.positions, freq, 2 * freq.shape[0])
+    k = k * d ** -0.5
+    cu, slots = step.cu_q_lens.tolist(), step.state_slots.tolist()
+    o = torch.zeros(t, h, e)
+    for b in range(len(slots)):
+        s = state[slots[b]].view(h, d, e).clone() if slots[b] else torch.zeros(h, d, e)
+        for i in range(cu[b], cu[b + 1]):
+            s = decay[:, None, None] * s + k[i][:, :, None] * v[i][:, None, :]
+            o[i] = torch.einsum("hde,hd->he", s, q[i])
+        if slots[b]:
+            state[slots[b]] = s.reshape(-1)
+    o = (o / torch.sqrt(o.square().mean(-1, keepdim=True) + norm_eps)).reshape(t, h * e)
+    return (o * (g * torch.sigmoid(g))).to(out_dtype)
+
+
+def routed_experts(x, ids, weights, w_gate_up, w_down, shared, logits, shared_gate_col, out_dtype, limited=None):
     t, w = x.shape
+    if hasattr(ids, "table"):               # a table's choice by token id
+        weight, ids = ids.weight, ids.table[ids.token_ids.long()[:t]]
+        weights = torch.full(ids.shape, weight)
     f = w_gate_up.shape[1] // 2
     out = torch.zeros(t, w)
     for i in range(t):
         for j in range(ids.shape[1]):
             e = int(ids[i, j])
             gu = w_gate_up[e].float() @ x[i].float()
-            hdn = (gu[:f] * torch.sigmoid(gu[:f]) * gu[f:]).to(x.dtype).float()
+            if limited is None:
+                hdn = gu[:f] * torch.sigmoid(gu[:f]) * gu[f:]
+            else:
+                a, b = gu[:f].clamp(max=limited[0]), gu[f:].clamp(-limited[0], limited[0])
+                hdn = a * torch.sigmoid(limited[1] * a) * (b + 1.0)
+            hdn = hdn.to(x.dtype).float()
             out[i] += weights[i, j] * (w_down[e].float() @ hdn)
     if shared is not None and shared_gate_col < 0:
         out = out + _plain(shared)
@@ -609,7 +649,7 @@ def routed_experts(x, ids, weights, w_gate_up, w_down, shared, logits, shared_ga
     return out
 
 
-ALL = ("state_space", "scale_", "stream_read", "gated_delta_rule", "gated_linear_recurrence", "route_experts", "routed_experts",
+ALL = ("retention", "squared_relu", "squared_relu_linear", "state_space", "scale_", "stream_read", "gated_delta_rule", "gated_linear_recurrence", "route_experts", "routed_experts",
        "embedding_scaled", "stream_add_", "limited_gate", "attn_prepare", "latent_prepare", "heads_linear",
        "masked_attention", "embedding_positions", "stream_rms_norm", "xielu", "softcap_", "qkv_bias_cache", "sigmoid_attention",
        "delta_rule", "patch_token_ids", "embedding", "rms_norm", "add_rms_norm", "qk_norm_rope_cache", "reshape_and_cache",
