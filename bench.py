@@ -403,8 +403,48 @@ def bovitar_like(q, layers: int, taps: int, softcap: float, state: int, ssm_grou
         "norm": {"eps": 1e-6}, "logit_scale": 0.5, "layers": entries})
 
 
+NEDUPEL_SIZES = {
+    # name -> the Nedupel sizes that go with the Qwen3 preset of DESIGN_SIZES[name]: latent layers of Zatirax's
+    # sizes, retention heads of 128 with values of 256 (twice the model's width in all at "8b"), and as many
+    # weights in a token's experts as in Qwen3's dense feed-forward
+    "0_6b": dict(rank=192, rot=64, r_heads=8, r_dim=128, r_vdim=256, experts=16, top=2, expert_ff=1536),
+    "8b": dict(rank=192, rot=64, r_heads=32, r_dim=128, r_vdim=256, experts=32, top=4, expert_ff=3072),
+}
+
+
+def nedupel_like(q, layers: int, rank: int, rot: int, r_heads: int, r_dim: int, r_vdim: int, experts: int, top: int,
+                 expert_ff: int):
+    """A Nedupel configuration with the layer sizes of the Qwen3 configuration ``q``: latent-attention and
+    retention layers in turn; the latent layers behind the first read its rows; the first feed-forward is
+    dense, the others are experts chosen by a table."""
+    from deterministic_inference_b200.config.nedupel_config import NedupelConfig
+    d = q.head_dim
+    entries = []
+    for i in range(layers):
+        mlp = {"kind": "dense", "ff": q.intermediate_size * 3 // 2} if i == 0 else \
+            {"kind": "moe", "expert": {"ff": expert_ff, "limit": 7.0}, "router": {"experts": experts, "top": top}}
+        if i % 2 == 0:
+            m = {"heads": q.num_attention_heads, "dim": d - rot, "rot_dim": rot, "vdim": d, "kv_rank": rank,
+                 "scale": d ** -0.5, "rot": {"base": 500000.0, "dims": rot,
+                                             "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+            if i:
+                m["kv_from"] = 0
+            entries.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
+        else:
+            entries.append({"type": "retention", "mlp": mlp,
+                            "mixer": {"heads": r_heads, "dim": r_dim, "vdim": r_vdim,
+                                      "decay": [1.0 - 2.0 ** (-5 - 8.0 * h / r_heads) for h in range(r_heads)],
+                                      "rot": {"base": 10000.0, "dims": r_dim}}})
+    return NedupelConfig.from_dict({
+        "architecture": "Nedupel", "vocab": q.vocab_size, "width": q.hidden_size, "max_positions": 8192,
+        "norm": {"eps": 1e-6}, "embedding": {"scale": 4.0}, "residual_mult": 0.25, "logit_scale": 0.5,
+        "layers": entries})
+
+
 def design_arm(a) -> int:
-    """``--design zatirax``: the same for the Zatirax design; ``--design kipezen``: for the Kipezen design,
+    """``--design nedupel``: the Nedupel design beside Zatirax (the closest: latent attention, a float32
+    stream), its kernels also beside the state-space recurrence and the routed experts of the other designs.
+    ``--design zatirax``: the same for the Zatirax design; ``--design kipezen``: for the Kipezen design,
     beside Gamilorn (the closest design) instead of Qwen3.  ``--design gamilorn``: prompt and decode throughput of the Gamilorn design at layer sizes of
     real models (random weights, ``--design-layers`` layers), beside Qwen3 at the same sizes, and
     the new design's kernels one by one beside the like kernels of Qwen3, each with its share of
@@ -885,6 +925,111 @@ def design_arm(a) -> int:
                     cache.release_slot(sl)
         return rows
 
+    def nedupel_kernel_rows(eng_n, eng_z, ncfg, zcfg):
+        """Nedupel's kernels on one layer's shapes and the like kernels of the other designs at equal sizes:
+        Zatirax's latent attention, stream kernel and feed-forward, the state-space recurrence of Bovitar, the
+        routed experts of Kipezen.  A prompt of ``n_prompt`` tokens, and a decode step of 8 requests with
+        ``ctx`` cached tokens."""
+        rows = {}
+        hbm, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+        lat, ret = ncfg.layers[0]["mixer"], ncfg.layers[1]["mixer"]
+        w, moe = ncfg.width, ncfg.layers[1]["mlp"]
+        lh, ld, lr, le, lc = lat["heads"], lat["dim"], lat["rot_dim"], lat["vdim"], lat["kv_rank"]
+        rh, rn, rp = ret["heads"], ret["dim"], ret["vdim"]
+        n_exp, top, eff = moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"]
+        win = zcfg.layers[1]["mixer"]["mask"]["size"]
+        bf = torch.bfloat16
+
+        def row(name, ms, nbytes, flops):
+            floor = max(nbytes / hbm, flops / tf) * 1e3
+            rows[name] = {"ms": round(ms, 4), "roofline_ms": round(floor, 4), "of_roofline": round(floor / ms, 4)}
+
+        for what, batch, q_len, before in (("prompt", 1, n_prompt, 0), ("decode_b8", 8, 1, ctx)):
+            t = batch * q_len
+            span = range(before, before + q_len)
+            x = torch.randn(t, w, device=dev).to(bf)
+            stream = torch.randn(t, w, device=dev)
+            one_w = torch.ones(w, device=dev)
+            for eng, label in ((eng_n, ""), (eng_z, "zatirax ")):
+                mine = not label
+                runner, cache = eng.runner, eng.cache
+                slots = [cache.allocate_slot() for _ in range(batch)]
+                if before:
+                    for sl in slots:
+                        runner.step([SequenceInput(sl, prompt_of(1000, before), 0, [])])
+                entries = [SequenceInput(sl, [1] * q_len, before, []) for sl in slots]
+                for e_ in entries:
+                    cache.allocate(e_.slot, before + q_len)
+                cache.reset_fresh_state()
+                step = build_step_batch(entries, cache, dev)
+                blocks = runner.model.blocks
+                mixer = blocks[0 if mine else 1].mixer
+                view = cache.view(0 if mine else 1, step)
+                ql = torch.randn(t, lh, lc + lr, device=dev).to(bf)
+                seen = (lambda p: p + 1) if mine else (lambda p: min(p + 1, win))
+                keys, held = batch * sum(seen(p) for p in span), seen(before + q_len - 1)
+                row(f"{what}: {label}latent attention ({'causal' if mine else 'window'})", timed(
+                    lambda: ops.masked_attention(ql, view.kv, view.attention_meta, (ld + lr) ** -0.5, 1, lc, view.page_size,
+                                                 "causal" if mine else "window", None if mine else win,
+                                                 values_in_keys=True)),
+                    2 * (t * lh * (2 * lc + lr) + batch * (lc + lr) * held), 2 * keys * lh * (2 * lc + lr))
+
+                def latent_rows(m, own, kind, amp):
+                    width = lh * (ld + lr) + (lc + lr if own else 0)
+                    lproj = torch.randn(t, width, device=dev).to(bf)
+
+                    def run():
+                        qq = ops.latent_prepare(lproj, lh, ld, lr, lc, m.latent_norm if own else None, 1e-6, m.freq,
+                                                step.positions, view.kv if own else None, view.slot_mapping,
+                                                view.page_size, bf, rotary_layout=kind, amplitude=amp)
+                        ops.heads_linear(lproj.as_strided((t, lh, ld), (width, ld + lr, 1)), m.w_key, qq[:, :, :lc])
+                        oo = torch.empty(t, lh, le, dtype=bf, device=dev)
+                        ops.heads_linear(ql[:, :, :lc], m.w_value, oo)
+                    return timed(run), 2 * (lproj.numel() + t * lh * (2 * lc + lr + le) + lh * lc * (ld + le)), \
+                        2 * t * lh * lc * (ld + le)
+                if mine:
+                    row(f"{what}: latent rows + the two products per head", *latent_rows(mixer, True, "pairs", 1.1))
+                    row(f"{what}: the same reading another layer's rows",
+                        *latent_rows(blocks[2].mixer, False, "pairs", 1.1))
+                    rproj = torch.randn(t, blocks[1].mixer.w_in.shape[0], device=dev).to(bf)
+                    rview = cache.view(1, step)
+                    row(f"{what}: retention (rotation, recurrence, norm, gate)", timed(lambda: ops.retention(
+                        rproj, blocks[1].mixer.decay, blocks[1].mixer.freq, rview.state, step, rh, rn, rp, 1e-6, bf)),
+                        rproj.numel() * 2 + t * rh * rp * 2 + batch * rh * rn * rp * 8, 4 * t * rh * rn * rp)
+                    # the state-space recurrence with as many heads and states of the same size
+                    inner, chan, heads = rh * rp, rh * rp + 2 * rh * rn, torch.zeros(rh, device=dev)
+                    sproj = torch.randn(t, inner + chan + rh, device=dev)
+                    sstate = torch.zeros(cache.max_reqs, rh * rn * rp + 3 * chan, device=dev)
+                    conv, norm = torch.randn(chan, 4, device=dev), torch.ones(inner, device=dev)
+                    row(f"{what}: state-space branch of the same heads and state", timed(lambda: ops.state_space(
+                        sproj, conv, None, heads, heads, heads, norm, sstate, step, rh, rp, rn, rh, 1, 4, 1e-6, bf)),
+                        batch * rh * rn * rp * 8 + t * (sproj.shape[1] * 4 + inner * 2), 5 * t * rh * rn * rp)
+                    row(f"{what}: scaled branch + add + norm of the float32 stream", timed(lambda: ops.stream_rms_norm(
+                        stream, one_w, 1e-6, bf, add=ops.WeightedSum([(0.25, x)]))), t * w * 12, 0)
+                    ff = blocks[0].feed_forward
+                    row(f"{what}: dense feed-forward, squared relu", timed(lambda: ff.forward(x)),
+                        2 * ff.intermediate_size * w * 2 + t * w * 4, 4 * t * ff.intermediate_size * w)
+                    ff = blocks[1].feed_forward
+                    ids = torch.randint(0, ncfg.vocab, (t,), generator=gen).to(torch.int32).to(dev)
+                    choice = ops.TableChoice(ids, ff.table, 1.0 / top)
+                    ex_bytes, ex_flops = min(n_exp, t * top) * eff * 3 * w * 2 + t * w * 6, 6 * t * top * eff * w
+                    row(f"{what}: experts of a table, limited gate", timed(lambda: ops.routed_experts(
+                        x, choice, None, ff.w_gate_up, ff.w_down, None, None, -1, bf, limited=ff.limited)), ex_bytes, ex_flops)
+                    given = ff.table[ids.long()].contiguous()
+                    share = torch.full(given.shape, 1.0 / top, device=dev)
+                    row(f"{what}: routed experts, silu gate (Kipezen's), the same choice", timed(lambda: ops.routed_experts(
+                        x, given, share, ff.w_gate_up, ff.w_down, None, None, -1, bf)), ex_bytes, ex_flops)
+                else:
+                    row(f"{what}: zatirax latent rows + the two products per head", *latent_rows(mixer, True, "halves", 1.0))
+                    row(f"{what}: zatirax post norm + add + norm of the float32 stream", timed(lambda: ops.stream_rms_norm(
+                        stream, one_w, 1e-6, bf, add=ops.NormedTerm(x, one_w, 1e-6))), t * w * 12, 0)
+                    ff = blocks[0].feed_forward
+                    row(f"{what}: zatirax dense feed-forward, limited gate", timed(lambda: ff.forward(x)),
+                        3 * ff.intermediate_size * w * 2 + t * w * 4, 6 * t * ff.intermediate_size * w)
+                for sl in slots:
+                    cache.release_slot(sl)
+        return rows
+
     sampler = ClockSampler()
     sampler.start()
     sizes = {}
@@ -900,6 +1045,11 @@ def design_arm(a) -> int:
             beside, bcfg = "gamilorn", gamilorn_like(qcfg, n_layers, **extra)
             extra = KIPEZEN_SIZES[name]
             gcfg = kipezen_like(qcfg, n_layers, **extra)
+        elif a.design == "nedupel":
+            # beside Zatirax, the closest design, at the same layer sizes
+            beside, bcfg = "zatirax", zatirax_like(qcfg, n_layers, **ZATIRAX_SIZES[name])
+            extra = NEDUPEL_SIZES[name]
+            gcfg = nedupel_like(qcfg, n_layers, **extra)
         elif a.design == "bovitar":
             # beside Kipezen, the closest design, at the same layer sizes
             beside, bcfg = "kipezen", kipezen_like(qcfg, n_layers, **KIPEZEN_SIZES[name])
@@ -921,14 +1071,14 @@ def design_arm(a) -> int:
                 r[f"decode_b{b}_tok_s"] = round(b / (dms / 1e3))
             out[label + "_result"] = r
         rows_of = {"zatirax": zatirax_kernel_rows, "kipezen": kipezen_kernel_rows,
-                   "bovitar": bovitar_kernel_rows}.get(a.design, kernel_rows)
+                   "bovitar": bovitar_kernel_rows, "nedupel": nedupel_kernel_rows}.get(a.design, kernel_rows)
         out["kernels"] = rows_of(engines[a.design], engines[beside], gcfg, bcfg)
         sizes[name] = out
         del engines
         import gc
         gc.collect()
         torch.cuda.empty_cache()
-    beside = {"kipezen": "gamilorn", "bovitar": "kipezen"}.get(a.design, "qwen3")
+    beside = {"kipezen": "gamilorn", "bovitar": "kipezen", "nedupel": "zatirax"}.get(a.design, "qwen3")
     print(json.dumps({"metric": f"{a.design} beside {beside} at equal layer sizes (bf16, 1 B200)", "impl": "ours",
                       "dtype": "bf16", "data": "synthetic, random weights", "n_gpus": 1,
                       "prompt_tokens": n_prompt, "decode_context": ctx, "decode_steps": a.point_steps,
@@ -963,8 +1113,8 @@ def main() -> int:
     ap.add_argument("--profile", default=None, choices=["decode", "prefill"],
                     help="bracket this region with cudaProfilerStart/Stop (for ncu "
                          "--profile-from-start off); the numbers of such a run are not a result")
-    ap.add_argument("--design", default=None, choices=["gamilorn", "zatirax", "kipezen", "bovitar"],
-                    help="measure this design beside Qwen3 (kipezen: beside Gamilorn; bovitar: beside Kipezen) at equal layer sizes instead of the default "
+    ap.add_argument("--design", default=None, choices=["gamilorn", "zatirax", "kipezen", "bovitar", "nedupel"],
+                    help="measure this design beside Qwen3 (kipezen: beside Gamilorn; bovitar: beside Kipezen; nedupel: beside Zatirax) at equal layer sizes instead of the default "
                          "workload (prints a line of its own)")
     ap.add_argument("--design-sizes", default="0_6b,8b", help=f"of {sorted(DESIGN_SIZES)}")
     ap.add_argument("--design-layers", type=int, default=4)
