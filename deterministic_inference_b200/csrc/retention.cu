@@ -202,7 +202,7 @@ __global__ void __launch_bounds__(256)
 retention_rotate_kernel(const __nv_bfloat16* proj, long long row_width, const float* __restrict__ freq, int rot,
                         const int* __restrict__ positions, int t_first, __nv_bfloat16* planes, long long plane,
                         int H, int N, float k_scale) {
-  extern __shared__ float cs[];            // cosines [rot / 2], sines [rot / 2]
+  extern __shared__ __align__(16) float cs[];            // cosines [rot / 2], sines [rot / 2]
   pdl_prologue(proj);
   const int tl = blockIdx.x, t = t_first + tl, half = rot >> 1;
   const float pos = (float)positions[t];
@@ -214,6 +214,33 @@ retention_rotate_kernel(const __nv_bfloat16* proj, long long row_width, const fl
   __syncthreads();
   const int HN = H * N;
   const __nv_bfloat16* x = proj + (long long)t * row_width;
+  if (rot == N && (half & 1) == 0) {
+    // the whole head turns: a thread takes two neighbouring pairs
+    const int per = half >> 1;
+    for (int i = threadIdx.x; i < 2 * H * per; i += 256) {
+      const int head = i / per, d = (i - head * per) * 2;           // heads of q, then of k
+      const __nv_bfloat16* src = x + (long long)head * N + d;
+      const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src));
+      const float2 w = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src + half));
+      const float2 c = *reinterpret_cast<const float2*>(cs + d), s = *reinterpret_cast<const float2*>(cs + half + d);
+      float a0 = __fmaf_rn(u.x, c.x, -__fmul_rn(w.x, s.x)), a1 = __fmaf_rn(u.y, c.y, -__fmul_rn(w.y, s.y));
+      float b0 = __fmaf_rn(w.x, c.x, __fmul_rn(u.x, s.x)), b1 = __fmaf_rn(w.y, c.y, __fmul_rn(u.y, s.y));
+      const bool is_k = head >= H;
+      if (is_k) {
+        a0 = __fmul_rn(a0, k_scale); a1 = __fmul_rn(a1, k_scale);
+        b0 = __fmul_rn(b0, k_scale); b1 = __fmul_rn(b1, k_scale);
+      }
+      __nv_bfloat16* dst = planes + (is_k ? 2 * plane : 0) + (long long)tl * HN + (long long)(is_k ? head - H : head) * N + d;
+      unsigned hi, lo;
+      split2(a0, a1, hi, lo);
+      *reinterpret_cast<unsigned*>(dst) = hi;
+      *reinterpret_cast<unsigned*>(dst + plane) = lo;
+      split2(b0, b1, hi, lo);
+      *reinterpret_cast<unsigned*>(dst + half) = hi;
+      *reinterpret_cast<unsigned*>(dst + plane + half) = lo;
+    }
+    return;
+  }
   for (int i = threadIdx.x * 2; i < 2 * HN; i += 512) {       // two neighbouring elements of one head
     const bool is_k = i >= HN;
     const int d = i % N;
@@ -327,52 +354,57 @@ retention_chunk_kernel(const __nv_bfloat16* planes, long long plane, const __nv_
   }
 }
 
-// grid (ceil(N P / 1024), H, B), a thread per 4 elements of a state.  In place: where a chunk's sum lay,
-// the state in front of the chunk, four elements as four hi (8 bytes) and four lo (8 bytes).
-__global__ void __launch_bounds__(256)
-retention_chain_kernel(float4* chunks, const float* __restrict__ decay, float* state, long long slot_stride,
-                       const int* __restrict__ cu, const int* __restrict__ state_slots, int H, int NP4) {
+// grid (N P / 256, H, B), a thread per 2 elements of a state.  In place: where a chunk's sum lay, the state
+// in front of the chunk, four elements as four hi (8 bytes) and four lo (8 bytes); a warp has read its
+// groups of four before it writes them.
+__global__ void __launch_bounds__(128)
+retention_chain_kernel(float2* chunks, const float* __restrict__ decay, float* state, long long slot_stride,
+                       const int* __restrict__ cu, const int* __restrict__ state_slots, int H, int NP2) {
   pdl_prologue(chunks, state);
-  const int i = blockIdx.x * 256 + threadIdx.x, h = blockIdx.y, b = blockIdx.z;
+  const int i = blockIdx.x * 128 + threadIdx.x, h = blockIdx.y, b = blockIdx.z;      // (NP2 is a multiple of 128)
   const int len = cu[b + 1] - cu[b];
-  if (i >= NP4 || len <= 0) return;
+  if (len <= 0) return;
   const long long slot = state_slots[b];
-  float4* srow = reinterpret_cast<float4*>(state + slot * slot_stride) + (long long)h * NP4;
-  float4 S = slot != 0 ? srow[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+  float2* srow = reinterpret_cast<float2*>(state + slot * slot_stride) + (long long)h * NP2;
+  float2 S = slot != 0 ? srow[i] : make_float2(0.f, 0.f);
   const float d = decay[h], d_chunk = powf(d, (float)CH);
   const int n_chunks = (len + CH - 1) / CH, place = first_place(cu, b);
-  constexpr int AHEAD = 4;
+  const int hi_at = (i >> 1) * 4 + (i & 1);             // in 4-byte words of a state
+  constexpr int AHEAD = 16;          // chunks whose loads are issued before the first is used
   for (int c0 = 0; c0 < n_chunks; c0 += AHEAD) {
-    float4 add[AHEAD];
+    float2 add[AHEAD];
 #pragma unroll
     for (int u = 0; u < AHEAD; ++u)
-      if (c0 + u < n_chunks) add[u] = chunks[((long long)(place + c0 + u) * H + h) * NP4 + i];
+      if (c0 + u < n_chunks) add[u] = chunks[((long long)(place + c0 + u) * H + h) * NP2 + i];
+    __syncwarp();
 #pragma unroll
     for (int u = 0; u < AHEAD; ++u)
       if (c0 + u < n_chunks) {
-        uint4 o;
-        split2(S.x, S.y, o.x, o.z);
-        split2(S.z, S.w, o.y, o.w);
-        reinterpret_cast<uint4*>(chunks)[((long long)(place + c0 + u) * H + h) * NP4 + i] = o;
+        unsigned hi, lo;
+        split2(S.x, S.y, hi, lo);
+        unsigned* dst = reinterpret_cast<unsigned*>(chunks + ((long long)(place + c0 + u) * H + h) * NP2);
+        dst[hi_at] = hi;
+        dst[hi_at + 2] = lo;
         const int left = len - (c0 + u) * CH;
         const float f = left >= CH ? d_chunk : powf(d, (float)left);
         S.x = __fmaf_rn(f, S.x, add[u].x);
         S.y = __fmaf_rn(f, S.y, add[u].y);
-        S.z = __fmaf_rn(f, S.z, add[u].z);
-        S.w = __fmaf_rn(f, S.w, add[u].w);
       }
   }
   if (slot != 0) srow[i] = S;
 }
 
-// grid (places, H), four warps of 16 tokens each, all P columns.
-template <int NPT>
-__global__ void __launch_bounds__(128)
+// grid (places, H), HALVES times four warps: a warp has 16 tokens and NPT * 64 of the columns (wide heads
+// are cut in two, which keeps more warps on an SM; both halves' warps make the same token weights).
+template <int NPT, int HALVES>
+__global__ void __launch_bounds__(128 * HALVES, 2)
 retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv_bfloat16* proj, long long row_width,
                         const unsigned char* chunks, const float* __restrict__ decay, const int* __restrict__ cu, int B,
                         int t_first, __nv_bfloat16* out, int H, int N, int P, float eps) {
   extern __shared__ __align__(16) unsigned char ro_smem[];
   __shared__ float pw[CH + 1];
+  __shared__ float squares[2][CH];
+  constexpr int OT = 128 * HALVES;
   pdl_prologue(planes, proj, chunks);
   int b, first, count;
   if (!chunk_at(cu, B, blockIdx.x, b, first, count)) return;
@@ -387,7 +419,7 @@ retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv
   __nv_bfloat16* Ss = Kh;                                            // [2][hi, lo][SR][vs]
   const int t0 = cu[b] + first;
   const int nv = N / 8, pv = P / 8;
-  for (int idx = threadIdx.x; idx < CH * nv; idx += 128) {
+  for (int idx = threadIdx.x; idx < CH * nv; idx += OT) {
     const int j = idx / nv, c = (idx - j * nv) * 8;
     const bool ok = j < count;
     const __nv_bfloat16* src = planes + (long long)(t0 - t_first + (ok ? j : 0)) * H * N + (long long)h * N + c;
@@ -396,7 +428,7 @@ retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv
     copy16(Kh + j * qs + c, src + 2 * plane, ok);
     copy16(Kl + j * qs + c, src + 3 * plane, ok);
   }
-  for (int idx = threadIdx.x; idx < CH * pv; idx += 128) {
+  for (int idx = threadIdx.x; idx < CH * pv; idx += OT) {
     const int j = idx / pv, c = (idx - j * pv) * 8;
     const bool ok = j < count;
     copy16(Vs + j * vs + c, proj + (long long)(ok ? t0 + j : t0) * row_width + 2ll * H * N + (long long)h * P + c, ok);
@@ -405,9 +437,10 @@ retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv
   if (threadIdx.x <= CH) pw[threadIdx.x] = powf(decay[h], (float)threadIdx.x);
   __pipeline_wait_prior(0);
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
-  const int m0 = warp * 16;
-  const bool active = m0 < count;
+  const int warp = (threadIdx.x >> 5) & 3, half = threadIdx.x >> 7;
+  const int lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+  const int m0 = warp * 16, p0 = half * NPT * 64;          // the warp's first token and column
+  const bool active = m0 < count && p0 < P;
 
   // q_i . k_j of the warp's 16 tokens and the chunk's tokens up to them
   float s[CH / 8][4];
@@ -450,7 +483,7 @@ retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv
   const unsigned char* src = chunks + ((long long)blockIdx.x * H + h) * N * P * 4;
   auto stage = [&](int kk, int buf) {
     __nv_bfloat16* hi = Ss + (size_t)buf * 2 * SR * vs;
-    for (int idx = threadIdx.x; idx < SR * (P / 4); idx += 128) {
+    for (int idx = threadIdx.x; idx < SR * (P / 4); idx += OT) {
       const int r = idx / (P / 4), c = idx - r * (P / 4);
       const unsigned char* p = src + ((long long)(kk * SR + r) * P + c * 4) * 4;
       __pipeline_memcpy_async(hi + r * vs + c * 4, p, 8);
@@ -477,8 +510,8 @@ retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv
       ldsm_x4(l0, l1, l2, l3, Ql + q_at + kk * 16);
 #pragma unroll
       for (int np = 0; np < NPT * 4; ++np)
-        if (np * 16 < P) {
-          const int at = ((lane & 7) + ((lane >> 3) & 1) * 8) * vs + np * 16 + (lane >> 4) * 8;
+        if (p0 + np * 16 < P) {
+          const int at = ((lane & 7) + ((lane >> 3) & 1) * 8) * vs + p0 + np * 16 + (lane >> 4) * 8;
           unsigned b0, b1, b2, b3, c0, c1, c2, c3;
           ldsm_x4_trans(b0, b1, b2, b3, sh + at);
           ldsm_x4_trans(c0, c1, c2, c3, sh + SR * vs + at);
@@ -492,7 +525,6 @@ retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv
     }
     __syncthreads();         // the stage is written again two steps on
   }
-  if (!active) return;
   const float f0 = pw[m0 + gid + 1], f1 = pw[m0 + gid + 9];
 #pragma unroll
   for (int n = 0; n < NPT * 8; ++n) {
@@ -501,12 +533,12 @@ retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv
   }
 #pragma unroll
   for (int kk = 0; kk < CH / 16; ++kk)
-    if (kk <= warp) {
+    if (active && kk <= warp) {
 #pragma unroll
       for (int np = 0; np < NPT * 4; ++np)
-        if (np * 16 < P) {
+        if (p0 + np * 16 < P) {
           unsigned b0, b1, b2, b3;
-          ldsm_x4_trans(b0, b1, b2, b3, Vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * vs + np * 16 + (lane >> 4) * 8);
+          ldsm_x4_trans(b0, b1, b2, b3, Vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * vs + p0 + np * 16 + (lane >> 4) * 8);
           mma_bf16(o[2 * np], wh[2 * kk][0], wh[2 * kk][1], wh[2 * kk + 1][0], wh[2 * kk + 1][1], b0, b1);
           mma_bf16(o[2 * np + 1], wh[2 * kk][0], wh[2 * kk][1], wh[2 * kk + 1][0], wh[2 * kk + 1][1], b2, b3);
           mma_bf16(o[2 * np], wl[2 * kk][0], wl[2 * kk][1], wl[2 * kk + 1][0], wl[2 * kk + 1][1], b0, b1);
@@ -516,21 +548,28 @@ retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv
   float ss[2] = {0.f, 0.f};
 #pragma unroll
   for (int n = 0; n < NPT * 8; ++n)
-    if (n * 8 < P)
+    if (p0 + n * 8 < P)
 #pragma unroll
       for (int r = 0; r < 2; ++r) ss[r] = __fmaf_rn(o[n][2 * r + 1], o[n][2 * r + 1], __fmaf_rn(o[n][2 * r], o[n][2 * r], ss[r]));
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], 1);
     ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], 2);
+    if (HALVES == 2 && tig == 0) squares[half][m0 + gid + 8 * r] = ss[r];
+  }
+  if (HALVES == 2) __syncthreads();       // a token's squares: the first half's columns, then the second's
+  if (!active) return;
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
     const int i = m0 + gid + 8 * r;
     if (i >= count) continue;
-    const float rstd = 1.0f / sqrtf(ss[r] / (float)P + eps);
+    const float total = HALVES == 2 ? __fadd_rn(squares[0][i], squares[1][i]) : ss[r];
+    const float rstd = 1.0f / sqrtf(total / (float)P + eps);
     const long long row = (long long)(t0 + i) * row_width + 2ll * H * N + (long long)H * P + (long long)h * P;
     __nv_bfloat16* dst = out + (long long)(t0 + i) * H * P + (long long)h * P;
 #pragma unroll
     for (int n = 0; n < NPT * 8; ++n) {
-      const int col = n * 8 + tig * 2;
+      const int col = p0 + n * 8 + tig * 2;
       if (col < P) {
         const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(proj + row + col));
         *reinterpret_cast<unsigned*>(dst + col) = pack_bf16(o[n][2 * r] * rstd * (g.x * sigmoid_f32(g.x)),
@@ -542,7 +581,7 @@ retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv
 
 constexpr int MOST_SMEM = 224 * 1024;
 
-template <int NPT>
+template <int NPT, int OUT_NPT, int HALVES>
 int launch_chunks(const __nv_bfloat16* planes, long long plane, const __nv_bfloat16* proj, long long row_width,
                   const float* decay, float* chunks, float* state, long long slot_stride, const int* cu,
                   const int* state_slots, int B, int t_first, int places, __nv_bfloat16* out, int H, int N, int P,
@@ -554,17 +593,20 @@ int launch_chunks(const __nv_bfloat16* planes, long long plane, const __nv_bfloa
   static DeviceOnce once;
   if (!once.done()) {
     if (cudaFuncSetAttribute(retention_chunk_kernel<NPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST_SMEM) != cudaSuccess ||
-        cudaFuncSetAttribute(retention_output_kernel<NPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST_SMEM) != cudaSuccess)
+        cudaFuncSetAttribute(retention_output_kernel<OUT_NPT, HALVES>, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST_SMEM) != cudaSuccess)
       return DIB_LAUNCH_FAILED;
+    // (as much of an SM's memory as shared memory as there is, so that two blocks of wide heads fit)
+    cudaFuncSetAttribute(retention_chunk_kernel<NPT>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
+    cudaFuncSetAttribute(retention_output_kernel<OUT_NPT, HALVES>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
     once.mark();
   }
   dib_launch(retention_chunk_kernel<NPT>, dim3(places, H, (N + 63) / 64), dim3(128), smem_c, st, planes, plane, proj,
              row_width, decay, cu, B, t_first, chunks, H, N, P);
   DIB_CHECK_LAUNCH();
-  dib_launch(retention_chain_kernel, dim3((N * P / 4 + 255) / 256, H, B), dim3(256), 0, st, (float4*)chunks, decay, state,
-             slot_stride, cu, state_slots, H, N * P / 4);
+  dib_launch(retention_chain_kernel, dim3(N * P / 256, H, B), dim3(128), 0, st, (float2*)chunks, decay, state,
+             slot_stride, cu, state_slots, H, N * P / 2);
   DIB_CHECK_LAUNCH();
-  dib_launch(retention_output_kernel<NPT>, dim3(places, H), dim3(128), smem_o, st, planes, plane, proj, row_width,
+  dib_launch(retention_output_kernel<OUT_NPT, HALVES>, dim3(places, H), dim3(128 * HALVES), smem_o, st, planes, plane, proj, row_width,
              (const unsigned char*)chunks, decay, cu, B, t_first, out, H, N, P, eps);
   DIB_CHECK_LAUNCH();
   return DIB_OK;
@@ -634,13 +676,13 @@ int dib_retention_chunked(const void* proj, long long row_width, const float* de
              (const __nv_bfloat16*)proj, row_width, freq, rot, positions, t_first, (__nv_bfloat16*)planes, plane, H, N,
              k_scale);
   DIB_CHECK_LAUNCH();
-#define DIB_RC(NPT)                                                                                                   \
-  return launch_chunks<NPT>((const __nv_bfloat16*)planes, plane, (const __nv_bfloat16*)proj, row_width, decay, chunks, state, \
+#define DIB_RC(NPT, OUT_NPT, HALVES)                                                                                  \
+  return launch_chunks<NPT, OUT_NPT, HALVES>((const __nv_bfloat16*)planes, plane, (const __nv_bfloat16*)proj, row_width, decay, chunks, state, \
                             slot_stride, cu, state_slots, B, t_first, places, (__nv_bfloat16*)out, H, N, P, eps, st)
-  if (P <= 64) DIB_RC(1);
-  if (P <= 128) DIB_RC(2);
-  if (P <= 192) DIB_RC(3);
-  DIB_RC(4);
+  if (P <= 64) DIB_RC(1, 1, 1);
+  if (P <= 128) DIB_RC(2, 1, 2);
+  if (P <= 192) DIB_RC(3, 2, 2);
+  DIB_RC(4, 2, 2);
 #undef DIB_RC
 }
 

@@ -235,17 +235,16 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ a_rows, const int* __re
   // this warp's column blocks: rows of B
   const int rows_b = mode == 0 ? 2 * N : N;
   const __nv_bfloat16* wb = w + (long long)expert * rows_b * K;
-  const int n0 = mode == 0 ? (blockIdx.y * 4 + warp) * (NJ / 2) * 8 : (blockIdx.y * 4 + warp) * NJ * 8;
+  constexpr int HALF = NJ / 2;
+  const int n0 = mode == 0 ? (blockIdx.y * 4 + warp) * HALF * 8 : (blockIdx.y * 4 + warp) * NJ * 8;
   const __nv_bfloat16* brow[NJ];
-  bool bok[NJ];
 #pragma unroll
   for (int j = 0; j < NJ; ++j) {
     int n;                 // the column of the output this thread's B row feeds
     long long rb;          // its row in B
-    if (mode == 0) { n = n0 + (j % (NJ / 2)) * 8 + g; rb = j < NJ / 2 ? n : (long long)N + n; }
+    if (mode == 0) { n = n0 + (j % HALF) * 8 + g; rb = j < HALF ? n : (long long)N + n; }
     else { n = n0 + j * 8 + g; rb = n; }
-    bok[j] = n < N;
-    brow[j] = wb + (bok[j] ? rb : 0) * K + tig * 8;
+    brow[j] = wb + (n < N ? rb : 0) * K + tig * 8;
   }
   float acc[MT][NJ][4];
 #pragma unroll
@@ -269,22 +268,32 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ a_rows, const int* __re
       *reinterpret_cast<uint4*>(As + r * as + c8 * 8) = v;
     }
     __syncthreads();
-    // (tiles of 16 rows are bound by the weight loads in flight: four steps' loads are issued ahead)
-#pragma unroll(MT == 1 ? 4 : 2)
-    for (int k = 0; k < kpad; k += 32) {
-      uint4 b[NJ];
-      const bool kin = k + tig * 8 < klen;
+    // The weight loads of AHEAD steps are issued before the first step's products (tiles of 16 rows are
+    // bound by the loads in flight).  No load has a condition: past the run's end it reads the row's
+    // first elements, which meet the zeros staged there.
+    constexpr int AHEAD = MT == 1 ? 16 / NJ : 2;
+    for (int k0 = 0; k0 < kpad; k0 += 32 * AHEAD) {
+      uint4 b[AHEAD][NJ];
 #pragma unroll
-      for (int j = 0; j < NJ; ++j)
-        b[j] = (bok[j] && kin) ? __ldg(reinterpret_cast<const uint4*>(brow[j] + kc + k)) : make_uint4(0, 0, 0, 0);
+      for (int u = 0; u < AHEAD; ++u) {
+        const int k = k0 + 32 * u, at = k + tig * 8 < klen ? kc + k : -tig * 8;
 #pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        const uint4 lo = *reinterpret_cast<const uint4*>(As + (m * 16 + g) * as + k + tig * 8);
-        const uint4 hi = *reinterpret_cast<const uint4*>(As + (m * 16 + g + 8) * as + k + tig * 8);
+        for (int j = 0; j < NJ; ++j) b[u][j] = __ldg(reinterpret_cast<const uint4*>(brow[j] + at));
+      }
 #pragma unroll
-        for (int j = 0; j < NJ; ++j) {
-          mma_bf16_16816(acc[m][j], lo.x, hi.x, lo.y, hi.y, b[j].x, b[j].y);
-          mma_bf16_16816(acc[m][j], lo.z, hi.z, lo.w, hi.w, b[j].z, b[j].w);
+      for (int u = 0; u < AHEAD; ++u) {
+        const int k = k0 + 32 * u;
+        if (k < kpad) {
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            const uint4 lo = *reinterpret_cast<const uint4*>(As + (m * 16 + g) * as + k + tig * 8);
+            const uint4 hi = *reinterpret_cast<const uint4*>(As + (m * 16 + g + 8) * as + k + tig * 8);
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) {
+              mma_bf16_16816(acc[m][j], lo.x, hi.x, lo.y, hi.y, b[u][j].x, b[u][j].y);
+              mma_bf16_16816(acc[m][j], lo.z, hi.z, lo.w, hi.w, b[u][j].z, b[u][j].w);
+            }
+          }
         }
       }
     }
@@ -299,11 +308,11 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ a_rows, const int* __re
       if (mode == 0) {
         __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + ((long long)tl * tile + r) * N;
 #pragma unroll
-        for (int j = 0; j < NJ / 2; ++j)
+        for (int j = 0; j < HALF; ++j)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             const int n = n0 + j * 8 + tig * 2 + e;
-            const float gt = acc[m][j][2 * hh + e], up = acc[m][j + NJ / 2][2 * hh + e];
+            const float gt = acc[m][j][2 * hh + e], up = acc[m][j + HALF][2 * hh + e];
             if (n < N) dst[n] = __float2bfloat16_rn(expert_gate(gt, up, limit, alpha));
           }
       } else {

@@ -30,6 +30,39 @@ __device__ __forceinline__ float source_load(const Source& s, long long i) {
   return v;
 }
 
+// The elements base + t, base + t + step, ... (N of them, those at or beyond base + width are 0) of a
+// source, every load of a split issued before the first is used; the splits are added in order.
+template <int N>
+__device__ __forceinline__ void source_load_strided(const Source& s, long long base, int t, int step, int width,
+                                                    float (&v)[N]) {
+  if (s.kind == 1) {
+    const __nv_bfloat16* p = reinterpret_cast<const __nv_bfloat16*>(s.p) + base;
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = t + i * step < width ? __bfloat162float(p[t + i * step]) : 0.f;
+    return;
+  }
+  const float* f = reinterpret_cast<const float*>(s.p) + base;
+#pragma unroll
+  for (int i = 0; i < N; ++i) v[i] = t + i * step < width ? f[t + i * step] : 0.f;
+  int k = 1;
+  for (; k + 4 <= s.splits; k += 4) {
+    float a[4][N];
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+#pragma unroll
+      for (int i = 0; i < N; ++i) a[u][i] = t + i * step < width ? f[(long long)(k + u) * s.stride + t + i * step] : 0.f;
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+#pragma unroll
+      for (int i = 0; i < N; ++i) v[i] = __fadd_rn(v[i], a[u][i]);
+  }
+  for (; k < s.splits; ++k) {
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+      if (t + i * step < width) v[i] = __fadd_rn(v[i], f[(long long)k * s.stride + t + i * step]);
+  }
+}
+
 // Store a float32 value as the dtype code says (0 float32, 1 bfloat16).
 __device__ __forceinline__ void store_as(void* p, int dtype, long long i, float v) {
   if (dtype == 1) reinterpret_cast<__nv_bfloat16*>(p)[i] = __float2bfloat16_rn(v);

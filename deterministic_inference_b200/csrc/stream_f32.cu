@@ -133,14 +133,51 @@ __global__ void limited_gate_kernel(Source gu, float limit, float alpha, void* o
 
 // One block per row.  TERMS > 0: residual[row] += a0 * x0[row] (+ a1 * x1[row]) first, the
 // terms added in their order; then out[row] = residual[row] / sqrt(mean(residual[row]^2) + eps)
-// * w.  The sum of squares is taken by a block of a width that depends on W alone.
-template <int TERMS>
+// * w.  The sum of squares is taken by a block of a width that depends on W alone, a thread's elements in
+// ascending order.  VPT > 0: a thread keeps its VPT elements of the row in registers (W <= VPT *
+// blockDim.x); the order of the sums is the same.
+template <int TERMS, int VPT>
 __global__ void stream_norm_kernel(float* residual, Source x0, float a0, Source x1, float a1,
                                    const float* w, void* out, int out_dtype, int W, float eps) {
   __shared__ float scratch[32];
-  pdl_prologue();
+  pdl_prologue(x0.p, x1.p, residual);
   const long long base = (long long)blockIdx.x * W;
   float ss = 0.f;
+  if (VPT > 0) {
+    constexpr int N = VPT > 0 ? VPT : 1;
+    float r[N], v[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      r[i] = c < W ? residual[base + c] : 0.f;
+    }
+    if (TERMS >= 1) {
+      source_load_strided<N>(x0, base, threadIdx.x, blockDim.x, W, v);
+#pragma unroll
+      for (int i = 0; i < N; ++i) r[i] = __fmaf_rn(a0, v[i], r[i]);
+    }
+    if (TERMS >= 2) {
+      source_load_strided<N>(x1, base, threadIdx.x, blockDim.x, W, v);
+#pragma unroll
+      for (int i = 0; i < N; ++i) r[i] = __fmaf_rn(a1, v[i], r[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < W) {
+        if (TERMS >= 1) residual[base + c] = r[i];
+        ss = __fmaf_rn(r[i], r[i], ss);
+      }
+    }
+    if (out == nullptr) return;
+    const float rstd = 1.0f / sqrtf(block_sum(ss, scratch) / (float)W + eps);
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < W) store_as(out, out_dtype, base + c, r[i] * rstd * w[c]);
+    }
+    return;
+  }
   for (int c = threadIdx.x; c < W; c += blockDim.x) {
     float r = residual[base + c];
     if (TERMS >= 1) r = __fmaf_rn(a0, source_load(x0, base + c), r);
@@ -325,9 +362,18 @@ int dib_stream_norm(float* residual, int terms, const void* x0, int kind0, int s
   if (out != nullptr && out_dtype != 0 && out_dtype != 1) return DIB_BAD_DTYPE;
   const Source s0 = make_source(x0, kind0, splits0, stride0), s1 = make_source(x1, kind1, splits1, stride1);
   const dim3 grid(rows), block(W >= 2048 ? 512 : (W >= 512 ? 256 : 128));
-  if (terms == 0) dib_launch(stream_norm_kernel<0>, grid, block, 0, st, residual, s0, a0, s1, a1, w, out, out_dtype, W, eps);
-  else if (terms == 1) dib_launch(stream_norm_kernel<1>, grid, block, 0, st, residual, s0, a0, s1, a1, w, out, out_dtype, W, eps);
-  else dib_launch(stream_norm_kernel<2>, grid, block, 0, st, residual, s0, a0, s1, a1, w, out, out_dtype, W, eps);
+  const int per_thread = (W + (int)block.x - 1) / (int)block.x;
+#define DIB_SN(TERMS, VPT) \
+  dib_launch(stream_norm_kernel<TERMS, VPT>, grid, block, 0, st, residual, s0, a0, s1, a1, w, out, out_dtype, W, eps)
+#define DIB_SNV(TERMS)                        \
+  if (per_thread <= 4) DIB_SN(TERMS, 4);      \
+  else if (per_thread <= 8) DIB_SN(TERMS, 8); \
+  else DIB_SN(TERMS, 0)
+  if (terms == 0) { DIB_SNV(0); }
+  else if (terms == 1) { DIB_SNV(1); }
+  else { DIB_SNV(2); }
+#undef DIB_SNV
+#undef DIB_SN
   DIB_CHECK_LAUNCH();
   return DIB_OK;
 }

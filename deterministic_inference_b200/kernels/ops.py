@@ -1680,8 +1680,9 @@ def heads_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> to
     m = x.shape[0]
     if x.dtype == torch.bfloat16 and m > HEADS_LINEAR_LIBRARY_ROWS:
         # many rows: the library's batched product, as for the other products of many rows
-        _launched(2)
-        out.transpose(0, 1).copy_(torch.bmm(x.transpose(0, 1), weight))
+        # (it writes rows of any stride itself)
+        _launched(1)
+        torch.bmm(x.transpose(0, 1), weight, out=out.transpose(0, 1))
         return out
     st = _lib("masked_attention").dib_heads_linear(
         _ptr(x), c_longlong(x.stride(0)), c_longlong(x.stride(1)), _ptr(weight), _ptr(out),
