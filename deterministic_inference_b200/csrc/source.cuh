@@ -31,8 +31,9 @@ __device__ __forceinline__ float source_load(const Source& s, long long i) {
 }
 
 // The elements base + t, base + t + step, ... (N of them, those at or beyond base + width are 0) of a
-// source, every load of a split issued before the first is used; the splits are added in order.
-template <int N>
+// source, the loads of AHEAD splits issued before the first is used; the splits are added in order (AHEAD 0:
+// the source is not split).
+template <int N, int AHEAD>
 __device__ __forceinline__ void source_load_strided(const Source& s, long long base, int t, int step, int width,
                                                     float (&v)[N]) {
   if (s.kind == 1) {
@@ -44,15 +45,17 @@ __device__ __forceinline__ void source_load_strided(const Source& s, long long b
   const float* f = reinterpret_cast<const float*>(s.p) + base;
 #pragma unroll
   for (int i = 0; i < N; ++i) v[i] = t + i * step < width ? f[t + i * step] : 0.f;
+  if (AHEAD == 0) return;
+  constexpr int U = AHEAD > 0 ? AHEAD : 1;
   int k = 1;
-  for (; k + 4 <= s.splits; k += 4) {
-    float a[4][N];
+  for (; k + U <= s.splits; k += U) {
+    float a[U][N];
 #pragma unroll
-    for (int u = 0; u < 4; ++u)
+    for (int u = 0; u < U; ++u)
 #pragma unroll
       for (int i = 0; i < N; ++i) a[u][i] = t + i * step < width ? f[(long long)(k + u) * s.stride + t + i * step] : 0.f;
 #pragma unroll
-    for (int u = 0; u < 4; ++u)
+    for (int u = 0; u < U; ++u)
 #pragma unroll
       for (int i = 0; i < N; ++i) v[i] = __fadd_rn(v[i], a[u][i]);
   }

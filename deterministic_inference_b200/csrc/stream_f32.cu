@@ -135,8 +135,9 @@ __global__ void limited_gate_kernel(Source gu, float limit, float alpha, void* o
 // terms added in their order; then out[row] = residual[row] / sqrt(mean(residual[row]^2) + eps)
 // * w.  The sum of squares is taken by a block of a width that depends on W alone, a thread's elements in
 // ascending order.  VPT > 0: a thread keeps its VPT elements of the row in registers (W <= VPT *
-// blockDim.x); the order of the sums is the same.
-template <int TERMS, int VPT>
+// blockDim.x); the order of the sums is the same.  AHEAD: splits whose loads are issued together (0 where no
+// term is split: fewer registers, more rows in flight).
+template <int TERMS, int VPT, int AHEAD>
 __global__ void stream_norm_kernel(float* residual, Source x0, float a0, Source x1, float a1,
                                    const float* w, void* out, int out_dtype, int W, float eps) {
   __shared__ float scratch[32];
@@ -152,12 +153,12 @@ __global__ void stream_norm_kernel(float* residual, Source x0, float a0, Source 
       r[i] = c < W ? residual[base + c] : 0.f;
     }
     if (TERMS >= 1) {
-      source_load_strided<N>(x0, base, threadIdx.x, blockDim.x, W, v);
+      source_load_strided<N, AHEAD>(x0, base, threadIdx.x, blockDim.x, W, v);
 #pragma unroll
       for (int i = 0; i < N; ++i) r[i] = __fmaf_rn(a0, v[i], r[i]);
     }
     if (TERMS >= 2) {
-      source_load_strided<N>(x1, base, threadIdx.x, blockDim.x, W, v);
+      source_load_strided<N, AHEAD>(x1, base, threadIdx.x, blockDim.x, W, v);
 #pragma unroll
       for (int i = 0; i < N; ++i) r[i] = __fmaf_rn(a1, v[i], r[i]);
     }
@@ -363,15 +364,19 @@ int dib_stream_norm(float* residual, int terms, const void* x0, int kind0, int s
   const Source s0 = make_source(x0, kind0, splits0, stride0), s1 = make_source(x1, kind1, splits1, stride1);
   const dim3 grid(rows), block(W >= 2048 ? 512 : (W >= 512 ? 256 : 128));
   const int per_thread = (W + (int)block.x - 1) / (int)block.x;
-#define DIB_SN(TERMS, VPT) \
-  dib_launch(stream_norm_kernel<TERMS, VPT>, grid, block, 0, st, residual, s0, a0, s1, a1, w, out, out_dtype, W, eps)
-#define DIB_SNV(TERMS)                        \
-  if (per_thread <= 4) DIB_SN(TERMS, 4);      \
-  else if (per_thread <= 8) DIB_SN(TERMS, 8); \
-  else DIB_SN(TERMS, 0)
-  if (terms == 0) { DIB_SNV(0); }
-  else if (terms == 1) { DIB_SNV(1); }
-  else { DIB_SNV(2); }
+  const bool split = (terms >= 1 && s0.splits > 1) || (terms >= 2 && s1.splits > 1);
+#define DIB_SN(TERMS, VPT, AHEAD) \
+  dib_launch(stream_norm_kernel<TERMS, VPT, AHEAD>, grid, block, 0, st, residual, s0, a0, s1, a1, w, out, out_dtype, W, eps)
+  // (wide rows without a split: the form that reads again has a third of the registers, so more rows in flight)
+#define DIB_SNV(TERMS, A4, A8)                    \
+  if (per_thread <= 4) DIB_SN(TERMS, 4, A4);      \
+  else if (A8 > 0 && per_thread <= 8) DIB_SN(TERMS, 8, (A8 > 0 ? A8 : 1)); \
+  else DIB_SN(TERMS, 0, 0)
+  if (terms == 0) { DIB_SNV(0, 0, 0); }
+  else if (terms == 1 && split) { DIB_SNV(1, 4, 2); }
+  else if (terms == 1) { DIB_SNV(1, 0, 0); }
+  else if (split) { DIB_SNV(2, 4, 2); }
+  else { DIB_SNV(2, 0, 0); }
 #undef DIB_SNV
 #undef DIB_SN
   DIB_CHECK_LAUNCH();
