@@ -5,8 +5,8 @@ sublayer's output times one constant (x <- x + m mixer(norm1(x)), then x <- x + 
 norms with weights stored around zero) and two kinds of mixer in any order: "latent_attention", causal
 softmax attention whose keys and values are rebuilt from a small latent per token, with a rotated key
 part shared by the heads (interleaved pairs, frequencies blended by pair index), where a layer may
-read the cached rows of an earlier one; and "retention", linear attention with a fixed decay per head,
-a per-head norm and a silu gate.  The feed-forward is dense with a squared relu, or a mixture of
+read the cached rows of an earlier one; and "retention", a matrix state per head that shrinks by
+one constant a token and is read without a softmax, behind it a per-head norm and a silu gate.  The feed-forward is dense with a squared relu, or a mixture of
 experts with limited gates whose choice is a table of the token ids.  The head has a matrix of its
 own; the logits are scaled by a constant.
 

@@ -1,4 +1,4 @@
-// Retention: linear attention with one fixed decay per head.
+// Retention: a matrix state per head that shrinks by one constant a token, read without a softmax.
 //
 // proj row (row_width elements): [q: H N | k: H N | v: H P | g: H P].  The first `rot` elements of
 // every q and k head turn in halves (element i with i + rot/2, angle = position * freq[i]); k is

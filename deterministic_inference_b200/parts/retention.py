@@ -1,12 +1,12 @@
-"""Retention: linear attention with one fixed decay per head, no softmax and no denominator.
+"""Retention: a matrix state per head that shrinks by one constant a token, read without a softmax.
 
 q = W_q x and k = W_k x (heads x ``head_dim``), v = W_v x and g = W_g x (heads x ``v_head_dim``), no
 biases, one product of the concatenated weights.  The position encoding rotates the first
 ``rotary_dim`` elements of every q and k head in halves (element i with i + rotary_dim / 2); k is
 multiplied by ``head_dim``^(-1/2) behind it.  Per head, with a state S [head_dim, v_head_dim] from zero:
     S <- decay_h S + k v^T;     o = S^T q.
-Each head's o is divided by its root mean square (``norm_eps``, no weight), the heads are
-concatenated, multiplied by silu(g) and projected by W_o.  The state is float32 and lives in the
+A head's output is o / sqrt(mean(o^2) + ``norm_eps``), without a weight; the heads side by side, times
+silu(g), go through W_o.  The state is float32 and lives in the
 request's state slot; the rotation, the decays, the recurrence and the norm are float32 whatever
 the engine's storage type.
 """

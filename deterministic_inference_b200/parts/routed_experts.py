@@ -2,8 +2,8 @@
 
 ``num_experts`` gated feed-forwards (W_down act(W_gate x, W_up x), no biases), of which each
 token uses ``top``.  ``activation`` "silu": silu(g) u; "limited_swish": with g = min(g, limit) and u =
-clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1).  ``score`` "table": no router; a stored table
-[vocabulary, top] of integers gives each token id its experts, each with weight ``route_scale`` / top.
+clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1).  ``score`` "table": no router; row i of a stored
+integer table [vocabulary, top] names the experts of token id i, all weighted ``route_scale`` / top.
 Otherwise, router: z = W_router x in float32, scores s = sigmoid(z) or (``score``
 "softmax") softmax(z) over all experts.  The choice is made on s + correction (a stored vector),
 the weights use s without it.  The experts form ``group_count`` equal groups of neighbours; a

@@ -9,8 +9,8 @@ bfloat16 engine stores (a yardstick for its tests); by default nothing is rounde
 The stream starts as embed[token] * s_e.  A layer is x <- x + m mixer(norm1(x)), then
 x <- x + m ff(norm2(x)), m one constant of the model, norms with weights around zero.  Mixers:
 "latent_attention" (keys and values from a small latent vector per token, a rotated key part
-shared by the heads; a layer may use the latents of an earlier one) and "retention" (linear
-attention with a fixed decay per head).  The feed-forward is dense with a squared relu, or a
+shared by the heads; a layer may use the latents of an earlier one) and "retention" (a matrix
+state per head that shrinks by a constant every token).  The feed-forward is dense with a squared relu, or a
 mixture of experts whose choice is a table of the token ids.
 """
 
