@@ -5,3 +5,4 @@ from .zatirax_config import ZatiraxConfig
 from .kipezen_config import KipezenConfig
 from .bovitar_config import BovitarConfig
 from .nedupel_config import NedupelConfig
+from .gikarax_config import GikaraxConfig

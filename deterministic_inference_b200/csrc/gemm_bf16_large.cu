@@ -338,10 +338,11 @@ __device__ __forceinline__ void store_rows_qkv(unsigned src, unsigned char* stag
 
 // What the epilogue applies.  GATED: limit > 0: g = min(gate, limit), u = clamp(up, -limit, limit),
 // g sigmoid(alpha g) (u + 1) of the float32 sums, the sigmoid on the special-function unit like
-// silu_gate's; else silu(gate) * up.  Otherwise: squared_relu: max(z, 0)^2 of the float32 sum.
+// silu_gate's; else silu(gate) * up.  Otherwise, of the float32 sum z: pointwise 1: max(z, 0)^2; 2: the
+// erf gelu z (1 + erf(z / sqrt 2)) / 2.
 struct Activation {
   float limit = 0.f, alpha = 0.f;
-  int squared_relu = 0;
+  int pointwise = 0;
 };
 __device__ __forceinline__ float gate_value(float g, float u, const Activation& act) {
   if (act.limit > 0.f) {
@@ -395,11 +396,17 @@ __device__ __forceinline__ void store_rows(unsigned src, const CUtensorMap* map_
         unsigned v[32];
         tc_ld32(src + col + h * 32, v);
         tc_wait_ld();
-        if (act.squared_relu) {
+        if (act.pointwise == 1) {
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
             const float z = fmaxf(__uint_as_float(v[e]), 0.f);
             v[e] = __float_as_uint(z * z);
+          }
+        } else if (act.pointwise == 2) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) {
+            const float z = __uint_as_float(v[e]);
+            v[e] = __float_as_uint(0.5f * z * (1.0f + erff(z * 0.70710678118654752f)));
           }
         }
 #pragma unroll
@@ -1008,7 +1015,7 @@ int dib_gemm_bf16_large_squared_relu(const void* x, const void* w, void* out, in
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) % 16 != 0)
     return DIB_BAD_ALIGN;
   Activation act;
-  act.squared_relu = 1;
+  act.pointwise = 1;
   const int shape = tile_shape(M, N, sm_count);
   if (shape == 2) return launch_pair<__nv_bfloat16, false, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, act);
   if (shape == 0) return launch_large<__nv_bfloat16, false, 128>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, nullptr, 1, act);
@@ -1032,7 +1039,8 @@ int dib_gemm_bf16_large_gated(const void* x, const void* w, void* out, int M, in
 // A product per tile of 128 rows with one of a stack of matrices: row tile m of x [M, K] (M a multiple
 // of 128) times matrix tile_matrix[m] of w.  gated = 0: w [matrices, N, K], out [M, N] bfloat16 or
 // float32 (N a multiple of 256).  gated = 1: w [matrices, 2N, K] (gate rows, then up rows), out [M, N]
-// bfloat16 = silu(gate) * up, or with limit > 0 the limited gate of gate_value (N a multiple of 128).  The table lies on the device and may be written
+// bfloat16 = silu(gate) * up, or with limit > 0 the limited gate of gate_value (N a multiple of 128).  gated = 2:
+// as 0 with the erf gelu of the product, bfloat16.  The table lies on the device and may be written
 // by the kernel before this one; it has M / 128 entries and one more, the number of row tiles in use
 // (the first ones; the rows of the others are left as they are).  Tiles of 128 x 256 by one CTA.
 int dib_gemm_bf16_large_grouped(const void* x, const void* w, void* out, int M, int N, int K, int gated, int out_fp32,
@@ -1040,16 +1048,17 @@ int dib_gemm_bf16_large_grouped(const void* x, const void* w, void* out, int M, 
                                 cudaStream_t st) {
   if (M == 0 || N == 0) return DIB_OK;
   if (K < 8 || K % 8 != 0 || sm_count < 1 || M % BM != 0 || matrices < 1 || tile_matrix == nullptr ||
-      N % (gated ? 128 : 256) != 0 || (gated && out_fp32))
+      N % (gated == 1 ? 128 : 256) != 0 || (gated && out_fp32) || gated < 0 || gated > 2)
     return DIB_BAD_SIZE;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) % 16 != 0)
     return DIB_BAD_ALIGN;
   Activation act;
   act.limit = limit;
   act.alpha = alpha;
-  if (gated) return launch_large<__nv_bfloat16, true, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, tile_matrix, matrices, act);
+  act.pointwise = gated == 2 ? 2 : 0;
+  if (gated == 1) return launch_large<__nv_bfloat16, true, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, tile_matrix, matrices, act);
   if (out_fp32) return launch_large<float, false, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, tile_matrix, matrices);
-  return launch_large<__nv_bfloat16, false, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, tile_matrix, matrices);
+  return launch_large<__nv_bfloat16, false, 256>(x, w, out, M, N, K, sm_count, st, QkvEpilogue{}, tile_matrix, matrices, act);
 }
 
 // The fused q/k/v projection of a prompt portion: x [M, K] times w [(Hq + 2 Hkv) * 128, K]^T,

@@ -35,14 +35,15 @@ __device__ __forceinline__ int first_visible(int pos, int mask_kind, int mask_si
 // One warp per (token, slot): slots 0 .. Hq-1 are query heads, then Hkv key heads, then Hkv value
 // heads of the projection row [q | k | v | ...] (row_width elements apart).  q and k: RMS norm
 // over the head with a weight (when given), then the first `rot` elements rotated by the token's
-// position: element i pairs with i + rot/2, angle = position * freq[i], all float32.
+// position: element i pairs with i + rot/2, angle = position * freq[i], cosine and sine times amp, all
+// float32.
 template <typename T>
 __global__ void __launch_bounds__(WARPS * 32)
 attn_prepare_kernel(Source proj, long long row_width, T* __restrict__ q_out, T* __restrict__ cache,
                     const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
                     const float* __restrict__ freq, int rot, const int* __restrict__ positions,
                     const int* __restrict__ slot_mapping, int T_tokens, int Hq, int Hkv, int D, int Dv,
-                    int page_size, long long num_pages) {
+                    int page_size, long long num_pages, float amp) {
   extern __shared__ float smem[];
   pdl_prologue(proj.p);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -88,7 +89,7 @@ attn_prepare_kernel(Source proj, long long row_width, T* __restrict__ q_out, T* 
     if (d < rot) {
       const int i = d < half ? d : d - half;
       const float a = __fmul_rn(pos, freq[i]);
-      const float c = cosf(a), sn = sinf(a);
+      const float c = __fmul_rn(amp, cosf(a)), sn = __fmul_rn(amp, sinf(a));
       v = d < half ? __fmaf_rn(x[d], c, -__fmul_rn(x[d + half], sn)) : __fmaf_rn(x[d], c, __fmul_rn(x[d - half], sn));
     }
     Elem<T>::store(dst + d, v);
@@ -99,7 +100,7 @@ attn_prepare_kernel(Source proj, long long row_width, T* __restrict__ q_out, T* 
 // A bias (float32 over [q | k | v]) joins the projection before anything else; the RMS norm of q and
 // of k runs per head (whole == 0, weights of D elements) or over all heads of the projection at once
 // (whole == 1, weights of Hq * D and Hkv * D elements); the rotation pairs element i with i + rot/2
-// (pairs == 0) or element 2i with 2i + 1 (pairs == 1), angle = position * freq[i].
+// (pairs == 0) or element 2i with 2i + 1 (pairs == 1), angle = position * freq[i], cosine and sine times amp.
 // cw given ([nq + nk + nv][taps] float32, the last tap the current token's): every channel of [q | k | v]
 // first passes a causal convolution over the sequence's tokens, y_t = sum_j cw[c][j] u_(t - taps + 1 + j),
 // with zeros before the sequence's start; the inputs before the step's first token come from the tail
@@ -115,7 +116,7 @@ attn_prepare_row_kernel(Source proj, long long row_width, const float* __restric
                         int D, int Dv, int page_size, long long num_pages, const float* __restrict__ cw, int taps,
                         const float* state, long long slot_stride, long long tail_at,
                         const int* __restrict__ token_seq, const int* __restrict__ cu_q_lens,
-                        const int* __restrict__ state_slots) {
+                        const int* __restrict__ state_slots, float amp) {
   extern __shared__ float smem[];      // the row's [q | k | v] (nq + nk + nv floats), then a factor per q and k head
   __shared__ float scratch[32];
   pdl_prologue(proj.p, state);
@@ -197,7 +198,7 @@ attn_prepare_row_kernel(Source proj, long long row_width, const float* __restric
       const bool first = pairs ? (d & 1) == 0 : d < half;
       const int other = pairs ? (d ^ 1) : (first ? d + half : d - half);
       const float a = __fmul_rn(pos, freq[pairs ? d >> 1 : (first ? d : d - half)]);
-      const float c = cosf(a), sn = sinf(a), o = x[s * D + other];
+      const float c = __fmul_rn(amp, cosf(a)), sn = __fmul_rn(amp, sinf(a)), o = x[s * D + other];
       v = first ? __fmaf_rn(v, c, -__fmul_rn(o, sn)) : __fmaf_rn(v, c, __fmul_rn(o, sn));
     }
     if (s < Hq) Elem<T>::store(q_out + (long long)t * nq + i, v);
@@ -268,6 +269,70 @@ latent_prepare_kernel(Source proj, long long row_width, T* __restrict__ q_out, T
   }
 }
 
+// ---- latent rows whose queries go through a latent of their own -----------------------------------
+// The projection row holds, at column q_at, a query latent of Cq elements, and at column kv_at the cached
+// latent of C elements and behind it a rotated key part of R (R may be 0).  One warp per (token, slot): slot 0
+// norms the cached latent (RMS, c_w) into the token's cache row [C + R] and rotates the key part; slot 1 norms
+// the query latent (RMS, q_w) into q_latent [T][Cq].
+template <typename T>
+__global__ void __launch_bounds__(WARPS * 32)
+latent_rows_kernel(Source proj, long long row_width, long long q_at, int Cq, const float* __restrict__ q_w,
+                   T* __restrict__ q_latent, long long kv_at, int C, int R, const float* __restrict__ c_w,
+                   T* __restrict__ cache, float eps, const float* __restrict__ freq, const int* __restrict__ positions,
+                   const int* __restrict__ slot_mapping, int T_tokens, int page_size, long long num_pages, int pairs,
+                   float amp) {
+  pdl_prologue(proj.p);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * WARPS + warp;
+  if (item >= 2ll * T_tokens) return;
+  const int t = (int)(item >> 1);
+  const bool query = (item & 1) != 0;
+  T* dst;
+  if (query) {
+    dst = q_latent + (long long)t * Cq;
+  } else {
+    if (cache == nullptr) return;
+    const int slot = slot_mapping[t];
+    if (slot < 0 || slot >= num_pages * page_size) return;
+    dst = cache + (long long)slot * (C + R);
+  }
+  const long long src = (long long)t * row_width + (query ? q_at : kv_at);
+  const int n = query ? Cq : C;
+  const float* w = query ? q_w : c_w;
+  constexpr int KEEP = 16;                   // elements of a lane kept in registers (the rest is read again)
+  float v[KEEP];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int d = lane + 32 * i;
+    v[i] = d < n ? round_to<T>(source_load(proj, src + d)) : 0.f;
+    ss = __fmaf_rn(v[i], v[i], ss);
+  }
+  for (int d = lane + 32 * KEEP; d < n; d += 32) {
+    const float x = round_to<T>(source_load(proj, src + d));
+    ss = __fmaf_rn(x, x, ss);
+  }
+  const float rstd = 1.0f / sqrtf(warp_sum(ss) / (float)n + eps);
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int d = lane + 32 * i;
+    if (d < n) Elem<T>::store(dst + d, v[i] * rstd * w[d]);
+  }
+  for (int d = lane + 32 * KEEP; d < n; d += 32)
+    Elem<T>::store(dst + d, round_to<T>(source_load(proj, src + d)) * rstd * w[d]);
+  if (query || R == 0) return;
+  const float pos = (float)positions[t];
+  const int half = R / 2;
+  for (int d = lane; d < R; d += 32) {
+    const bool first = pairs ? (d & 1) == 0 : d < half;
+    const float a = __fmul_rn(pos, freq[pairs ? d >> 1 : (first ? d : d - half)]);
+    const float c = __fmul_rn(amp, cosf(a)), sn = __fmul_rn(amp, sinf(a));
+    const float u = round_to<T>(source_load(proj, src + C + d));
+    const float o = round_to<T>(source_load(proj, src + C + (pairs ? (d ^ 1) : (first ? d + half : d - half))));
+    Elem<T>::store(dst + C + d, first ? __fmaf_rn(u, c, -__fmul_rn(o, sn)) : __fmaf_rn(u, c, __fmul_rn(o, sn)));
+  }
+}
+
 // ---- a product per head --------------------------------------------------------------------------
 // out[m, h, n] = sum_k x[m, h, k] * w[h, k, n]; x and out with free row and head strides (elements),
 // w contiguous [H, K, N].  float32 accumulation.  A block takes HL_ROWS rows and HL_COLS columns of one
@@ -327,7 +392,7 @@ masked_attention_kernel(const T* __restrict__ q, T* __restrict__ out, const T* _
                         const int* __restrict__ token_seq, const int* __restrict__ positions,
                         int T_tokens, int Hq, int Hkv, int Dk, int Dv, int Dv_stored, int page_size,
                         float scale, int mask_kind, int mask_size, int keep, const float* __restrict__ sink,
-                        Source gate, long long gate_row, long long gate_col, float softcap) {
+                        Source gate, long long gate_row, long long gate_col, int gate_heads, float softcap) {
   extern __shared__ float smem[];
   pdl_prologue(q, cache, block_table, token_seq, positions, gate.p);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -398,22 +463,23 @@ masked_attention_kernel(const T* __restrict__ q, T* __restrict__ out, const T* _
     if (d < Dv) {
       float o = acc[i] * inv;
       if (gate.p != nullptr)
-        o = round_to<T>(o) * sigmoid_f32(round_to<T>(source_load(gate, (long long)t * gate_row + gate_col + (long long)h * Dv + d)));
+        o = round_to<T>(o) * sigmoid_f32(round_to<T>(source_load(gate, (long long)t * gate_row + gate_col + (gate_heads ? h : (long long)h * Dv + d))));
       Elem<T>::store(orow + d, o);
     }
   }
 }
 
-// x[t, c] *= sigmoid(gate[t, gate_col + c]), in place; float32 arithmetic, one rounding
+// x[t, c] *= sigmoid(gate[t, gate_col + c / per]), in place; float32 arithmetic, one rounding (per: elements
+// that share a gate number)
 template <typename T>
 __global__ void sigmoid_gate_kernel(T* __restrict__ x, Source gate, long long gate_row, long long gate_col,
-                                    int rows, int width) {
+                                    int rows, int width, int per) {
   pdl_prologue(x, gate.p);
   const long long n = (long long)rows * width;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n;
        i += (long long)gridDim.x * blockDim.x) {
     const long long r = i / width, c = i % width;
-    const float g = round_to<T>(source_load(gate, r * gate_row + gate_col + c));
+    const float g = round_to<T>(source_load(gate, r * gate_row + gate_col + c / per));
     Elem<T>::store(x + i, Elem<T>::load(x + i) * sigmoid_f32(g));
   }
 }
@@ -423,13 +489,13 @@ int launch_masked_attention(const void* q, void* out, const void* cache, const i
                             int max_blocks, const int* token_seq, const int* positions, int T_tokens, int Hq,
                             int Hkv, int Dk, int Dv, int Dv_stored, int page_size, float scale, int mask_kind,
                             int mask_size, int keep, const float* sink, Source gate, long long gate_row,
-                            long long gate_col, float softcap, cudaStream_t st) {
+                            long long gate_col, int gate_heads, float softcap, cudaStream_t st) {
   const int blocks = ceil_div_host((long long)T_tokens * Hq, WARPS);
   const size_t smem = (size_t)WARPS * Dk * sizeof(float);
 #define DIB_MA(NV)                                                                                       \
   dib_launch(masked_attention_kernel<T, NV>, dim3(blocks), dim3(WARPS * 32), smem, st, (const T*)q, (T*)out, \
              (const T*)cache, block_table, max_blocks, token_seq, positions, T_tokens, Hq, Hkv, Dk, Dv,   \
-             Dv_stored, page_size, scale, mask_kind, mask_size, keep, sink, gate, gate_row, gate_col, softcap)
+             Dv_stored, page_size, scale, mask_kind, mask_size, keep, sink, gate, gate_row, gate_col, gate_heads, softcap)
   if (Dv <= 64) DIB_MA(2);
   else if (Dv <= 128) DIB_MA(4);
   else if (Dv <= 256) DIB_MA(8);
@@ -448,7 +514,7 @@ extern "C" {
 int dib_attn_prepare(const void* proj, int kind, int splits, long long stride, long long row_width, void* q_out,
                      void* cache, const float* q_w, const float* k_w, float eps, const float* freq, int rot,
                      const int* positions, const int* slot_mapping, int T, int Hq, int Hkv, int D, int Dv,
-                     int page_size, long long num_pages, int dtype, cudaStream_t st) {
+                     int page_size, long long num_pages, int dtype, float amp, cudaStream_t st) {
   if (T == 0) return DIB_OK;
   if (D < 1 || D > 2048 || Dv < 1 || Hq < 1 || Hkv < 1 || rot < 0 || rot > D || rot % 2 || page_size < 1)
     return DIB_BAD_SIZE;
@@ -458,11 +524,11 @@ int dib_attn_prepare(const void* proj, int kind, int splits, long long stride, l
   const size_t smem = (size_t)WARPS * D * sizeof(float);
   if (dtype == 0)
     dib_launch(attn_prepare_kernel<float>, dim3(blocks), dim3(WARPS * 32), smem, st, src, row_width, (float*)q_out,
-               (float*)cache, q_w, k_w, eps, freq, rot, positions, slot_mapping, T, Hq, Hkv, D, Dv, page_size, num_pages);
+               (float*)cache, q_w, k_w, eps, freq, rot, positions, slot_mapping, T, Hq, Hkv, D, Dv, page_size, num_pages, amp);
   else if (dtype == 1)
     dib_launch(attn_prepare_kernel<__nv_bfloat16>, dim3(blocks), dim3(WARPS * 32), smem, st, src, row_width,
                (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, q_w, k_w, eps, freq, rot, positions, slot_mapping, T,
-               Hq, Hkv, D, Dv, page_size, num_pages);
+               Hq, Hkv, D, Dv, page_size, num_pages, amp);
   else return DIB_BAD_DTYPE;
   DIB_CHECK_LAUNCH();
   return DIB_OK;
@@ -476,7 +542,7 @@ int dib_attn_prepare_row(const void* proj, int kind, int splits, long long strid
                          const int* slot_mapping, int T, int Hq, int Hkv, int D, int Dv, int page_size,
                          long long num_pages, int dtype, const float* cw, int taps, float* state,
                          long long slot_stride, long long tail_at, const int* token_seq, const int* cu_q_lens,
-                         const int* state_slots, int B, cudaStream_t st) {
+                         const int* state_slots, int B, float amp, cudaStream_t st) {
   if (T == 0) return DIB_OK;
   if (D < 1 || Dv < 1 || Hq < 1 || Hkv < 1 || rot < 0 || rot > D || rot % 2 || page_size < 1) return DIB_BAD_SIZE;
   if (cw != nullptr && (taps < 1 || taps > 64 || token_seq == nullptr || cu_q_lens == nullptr ||
@@ -496,7 +562,7 @@ int dib_attn_prepare_row(const void* proj, int kind, int splits, long long strid
     dib_launch(attn_prepare_row_kernel<float>, dim3(T), dim3(ROW_THREADS), smem, st, src, row_width, bias,
                (float*)q_out, (float*)cache, q_w, k_w, whole, eps, freq, rot, pairs, positions, slot_mapping, Hq, Hkv,
                D, Dv, page_size, num_pages, cw, taps, (const float*)state, slot_stride, tail_at, token_seq, cu_q_lens,
-               state_slots);
+               state_slots, amp);
   } else if (dtype == 1) {
     if (smem > 48 * 1024 && !once16.done()) {
       if (cudaFuncSetAttribute(attn_prepare_row_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -506,7 +572,7 @@ int dib_attn_prepare_row(const void* proj, int kind, int splits, long long strid
     dib_launch(attn_prepare_row_kernel<__nv_bfloat16>, dim3(T), dim3(ROW_THREADS), smem, st, src, row_width, bias,
                (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, q_w, k_w, whole, eps, freq, rot, pairs, positions,
                slot_mapping, Hq, Hkv, D, Dv, page_size, num_pages, cw, taps, (const float*)state, slot_stride, tail_at,
-               token_seq, cu_q_lens, state_slots);
+               token_seq, cu_q_lens, state_slots, amp);
   } else return DIB_BAD_DTYPE;
   DIB_CHECK_LAUNCH();
   if (cw != nullptr && taps > 1 && B > 0) {
@@ -540,6 +606,30 @@ int dib_latent_prepare(const void* proj, int kind, int splits, long long stride,
   return DIB_OK;
 }
 
+// R 0: no rotated key part (freq null).  cache null: nothing is stored.
+int dib_latent_rows(const void* proj, int kind, int splits, long long stride, long long row_width, long long q_at, int Cq,
+                    const float* q_w, void* q_latent, long long kv_at, int C, int R, const float* c_w, void* cache,
+                    float eps, const float* freq, const int* positions, const int* slot_mapping, int T, int page_size,
+                    long long num_pages, int dtype, int pairs, float amp, cudaStream_t st) {
+  if (T == 0) return DIB_OK;
+  if (Cq < 1 || C < 1 || R < 0 || R % 2 || (R > 0 && freq == nullptr) || page_size < 1 || q_at < 0 || kv_at < 0 ||
+      q_at + Cq > row_width || kv_at + C + R > row_width || q_w == nullptr || c_w == nullptr)
+    return DIB_BAD_SIZE;
+  const Source src = make_source(proj, kind, splits, stride);
+  const int blocks = ceil_div_host(2ll * T, WARPS);
+  if (dtype == 0)
+    dib_launch(latent_rows_kernel<float>, dim3(blocks), dim3(WARPS * 32), 0, st, src, row_width, q_at, Cq, q_w,
+               (float*)q_latent, kv_at, C, R, c_w, (float*)cache, eps, freq, positions, slot_mapping, T, page_size,
+               num_pages, pairs, amp);
+  else if (dtype == 1)
+    dib_launch(latent_rows_kernel<__nv_bfloat16>, dim3(blocks), dim3(WARPS * 32), 0, st, src, row_width, q_at, Cq, q_w,
+               (__nv_bfloat16*)q_latent, kv_at, C, R, c_w, (__nv_bfloat16*)cache, eps, freq, positions, slot_mapping, T,
+               page_size, num_pages, pairs, amp);
+  else return DIB_BAD_DTYPE;
+  DIB_CHECK_LAUNCH();
+  return DIB_OK;
+}
+
 int dib_heads_linear(const void* x, long long xs_m, long long xs_h, const void* w, void* out, long long os_m,
                      long long os_h, int M, int H, int K, int N, int dtype, cudaStream_t st) {
   if (M == 0) return DIB_OK;
@@ -563,17 +653,17 @@ int dib_heads_linear(const void* x, long long xs_m, long long xs_h, const void* 
 }
 
 int dib_sigmoid_gate_(void* x, const void* gate, int kind, int splits, long long stride, long long gate_row,
-                      long long gate_col, int rows, int width, int dtype, cudaStream_t st) {
+                      long long gate_col, int rows, int width, int per, int dtype, cudaStream_t st) {
   if (rows == 0) return DIB_OK;
-  if (width < 1) return DIB_BAD_SIZE;
+  if (width < 1 || per < 1) return DIB_BAD_SIZE;
   const Source g = make_source(gate, kind, splits, stride);
   const long long n = (long long)rows * width;
   const int blocks = (int)((n + 255) / 256 > 148 * 16 ? 148 * 16 : (n + 255) / 256);
   if (dtype == 0)
-    dib_launch(sigmoid_gate_kernel<float>, dim3(blocks), dim3(256), 0, st, (float*)x, g, gate_row, gate_col, rows, width);
+    dib_launch(sigmoid_gate_kernel<float>, dim3(blocks), dim3(256), 0, st, (float*)x, g, gate_row, gate_col, rows, width, per);
   else if (dtype == 1)
     dib_launch(sigmoid_gate_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, st, (__nv_bfloat16*)x, g, gate_row,
-               gate_col, rows, width);
+               gate_col, rows, width, per);
   else return DIB_BAD_DTYPE;
   DIB_CHECK_LAUNCH();
   return DIB_OK;
@@ -589,7 +679,7 @@ int dib_masked_attention_mma(const void* q, void* out, const void* cache, const 
                              int num_tiles, const float* sink, int Hq, int Hkv, int Dk, int Dv, int Dv_stored, int page_size,
                              float scale, int mask_kind, int mask_size, int keep, const void* gate, int gate_kind,
                              int gate_splits, long long gate_stride, long long gate_row, long long gate_col,
-                             int rows, float* partial_o, float* partial_ml, int chunk_tiles, int max_chunks,
+                             int gate_heads, int rows, float* partial_o, float* partial_ml, int chunk_tiles, int max_chunks,
                              int num_tokens, float softcap, cudaStream_t st) {
   if (num_tiles == 0) return DIB_OK;
   if (Dk < 16 || Dk % 16 || Dv < 16 || Dv % 16 || Dv > 256 || Hkv < 1 || Hq % Hkv != 0 || Hq / Hkv > rows ||
@@ -602,7 +692,7 @@ int dib_masked_attention_mma(const void* q, void* out, const void* cache, const 
 #define DIB_MAM(NV, ROWS)                                                                                    \
   return ma_mma::launch<NV, ROWS>(q, out, cache, block_table, max_blocks, positions, seq_lens, cu_q_lens, tiles, num_tiles, \
                                   sink, Hq, Hkv, Dk, Dv, Dv_stored, page_size, scale, mask_kind, mask_size, keep, g, \
-                                  gate_row, gate_col, partial_o, partial_ml, chunk_tiles, max_chunks, num_tokens, softcap, st)
+                                  gate_row, gate_col, gate_heads, partial_o, partial_ml, chunk_tiles, max_chunks, num_tokens, softcap, st)
   const int nv = (Dv + 63) / 64;
   if (rows == 64) {
     if (nv == 1) DIB_MAM(4, 64);
@@ -618,12 +708,12 @@ int dib_masked_attention_mma(const void* q, void* out, const void* cache, const 
 }
 
 // sink null: a plain softmax.  gate null: no output gate; else out *= sigmoid(gate[t, gate_col + h * Dv + d])
-// with rows gate_row elements apart.  Dv_stored 0: a key's first Dv elements are its value.
+// (gate_heads: gate[t, gate_col + h], one number per head) with rows gate_row elements apart.  Dv_stored 0: a key's first Dv elements are its value.
 int dib_masked_attention(const void* q, void* out, const void* cache, const int* block_table, int max_blocks,
                          const int* token_seq, const int* positions, int T, int Hq, int Hkv, int Dk, int Dv,
                          int Dv_stored, int page_size, float scale, int mask_kind, int mask_size, int keep,
                          const float* sink, const void* gate, int gate_kind, int gate_splits,
-                         long long gate_stride, long long gate_row, long long gate_col, int dtype, float softcap,
+                         long long gate_stride, long long gate_row, long long gate_col, int gate_heads, int dtype, float softcap,
                          cudaStream_t st) {
   if (T == 0) return DIB_OK;
   if (Dk < 1 || Dk > 2048 || Dv < 1 || Dv > 1024 || Hkv < 1 || Hq % Hkv != 0 || page_size < 1 ||
@@ -634,11 +724,11 @@ int dib_masked_attention(const void* q, void* out, const void* cache, const int*
   if (dtype == 0)
     return launch_masked_attention<float>(q, out, cache, block_table, max_blocks, token_seq, positions, T, Hq,
                                           Hkv, Dk, Dv, Dv_stored, page_size, scale, mask_kind, mask_size, keep, sink, g,
-                                          gate_row, gate_col, softcap, st);
+                                          gate_row, gate_col, gate_heads, softcap, st);
   if (dtype == 1)
     return launch_masked_attention<__nv_bfloat16>(q, out, cache, block_table, max_blocks, token_seq, positions, T,
                                                   Hq, Hkv, Dk, Dv, Dv_stored, page_size, scale, mask_kind,
-                                                  mask_size, keep, sink, g, gate_row, gate_col, softcap, st);
+                                                  mask_size, keep, sink, g, gate_row, gate_col, gate_heads, softcap, st);
   return DIB_BAD_DTYPE;
 }
 

@@ -62,7 +62,7 @@ masked_attention_mma_kernel(const __nv_bfloat16* q, __nv_bfloat16* out, const __
                             const int* cu_q_lens, const int* tiles, const float* sink, int Hq, int Hkv, int D,
                             int VD, int VD_stored,
                             int page_size, float scale, int mask_kind, int mask_size, int keep, Source gate,
-                            long long gate_row, long long gate_col, float* partial_o, float* partial_ml,
+                            long long gate_row, long long gate_col, int gate_heads, float* partial_o, float* partial_ml,
                             int chunk_tiles, int max_chunks, float softcap) {
   extern __shared__ __align__(16) unsigned char mam_smem[];
   const int R = Hq / Hkv;
@@ -299,9 +299,10 @@ masked_attention_mma_kernel(const __nv_bfloat16* q, __nv_bfloat16* out, const __
       if (col < VD) {
         float x0 = o[n][2 * h] * inv, x1 = o[n][2 * h + 1] * inv;
         if (gate.p != nullptr) {
-          const long long at = (long long)t * gate_row + gate_col + (long long)head * VD + col;
+          // (gate_heads: one number per head)
+          const long long at = (long long)t * gate_row + gate_col + (gate_heads ? head : (long long)head * VD + col);
           x0 = round_to<__nv_bfloat16>(x0) * sigmoid_f32(round_to<__nv_bfloat16>(source_load(gate, at)));
-          x1 = round_to<__nv_bfloat16>(x1) * sigmoid_f32(round_to<__nv_bfloat16>(source_load(gate, at + 1)));
+          x1 = round_to<__nv_bfloat16>(x1) * sigmoid_f32(round_to<__nv_bfloat16>(source_load(gate, gate_heads ? at : at + 1)));
         }
         *reinterpret_cast<__nv_bfloat162*>(dst + col) = __floats2bfloat162_rn(x0, x1);
       }
@@ -315,8 +316,8 @@ masked_attention_mma_kernel(const __nv_bfloat16* q, __nv_bfloat16* out, const __
 __global__ void masked_attention_merge_kernel(const float* partial_o, const float* partial_ml, __nv_bfloat16* out,
                                               const int* positions, const float* sink, int Hq, int VD,
                                               int mask_kind, int mask_size, int keep, Source gate,
-                                              long long gate_row, long long gate_col, int chunk_tiles,
-                                              int max_chunks) {
+                                              long long gate_row, long long gate_col, int gate_heads,
+                                              int chunk_tiles, int max_chunks) {
   pdl_prologue(partial_o, partial_ml, gate.p);
   const int t = blockIdx.x, h = blockIdx.y;
   const int pos = positions[t];
@@ -341,7 +342,7 @@ __global__ void masked_attention_merge_kernel(const float* partial_o, const floa
     v *= inv;
     if (gate.p != nullptr)
       v = round_to<__nv_bfloat16>(v) *
-          sigmoid_f32(round_to<__nv_bfloat16>(source_load(gate, (long long)t * gate_row + gate_col + (long long)h * VD + col)));
+          sigmoid_f32(round_to<__nv_bfloat16>(source_load(gate, (long long)t * gate_row + gate_col + (gate_heads ? h : (long long)h * VD + col))));
     out[row * VD + col] = __float2bfloat16_rn(v);
   }
 }
@@ -359,7 +360,7 @@ template <int NV16, int ROWS>
 static int launch(const void* q, void* out, const void* cache, const int* block_table, int bt_width,
                   const int* positions, const int* seq_lens, const int* cu_q_lens, const int* tiles, int num_tiles,
                   const float* sink, int Hq, int Hkv, int D, int VD, int VD_stored, int page_size, float scale, int mask_kind,
-                  int mask_size, int keep, Source gate, long long gate_row, long long gate_col, float* partial_o,
+                  int mask_size, int keep, Source gate, long long gate_row, long long gate_col, int gate_heads, float* partial_o,
                   float* partial_ml, int chunk_tiles, int max_chunks, int num_tokens, float softcap, cudaStream_t st) {
   const size_t smem = smem_bytes(D, VD, VD_stored, ROWS);
   if (smem > MAX_DYNAMIC_SMEM) return DIB_BAD_SIZE;
@@ -374,13 +375,13 @@ static int launch(const void* q, void* out, const void* cache, const int* block_
   dib_launch(masked_attention_mma_kernel<NV16, ROWS>, dim3(num_tiles, Hkv, chunked ? max_chunks : 1), dim3(ROWS * 2),
              smem, st, (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)cache, block_table,
              bt_width, positions, seq_lens, cu_q_lens, tiles, sink, Hq, Hkv, D, VD, VD_stored, page_size, scale, mask_kind,
-             mask_size, keep, gate, gate_row, gate_col, chunked ? partial_o : (float*)nullptr,
+             mask_size, keep, gate, gate_row, gate_col, gate_heads, chunked ? partial_o : (float*)nullptr,
              chunked ? partial_ml : (float*)nullptr, chunk_tiles, max_chunks, softcap);
   DIB_CHECK_LAUNCH();
   if (chunked) {
     dib_launch(masked_attention_merge_kernel, dim3(num_tokens, Hq), dim3(VD >= 128 ? 128 : 64), 0, st,
                (const float*)partial_o, (const float*)partial_ml, (__nv_bfloat16*)out, positions, sink, Hq, VD,
-               mask_kind, mask_size, keep, gate, gate_row, gate_col, chunk_tiles, max_chunks);
+               mask_kind, mask_size, keep, gate, gate_row, gate_col, gate_heads, chunk_tiles, max_chunks);
     DIB_CHECK_LAUNCH();
   }
   return DIB_OK;

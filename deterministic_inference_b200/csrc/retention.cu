@@ -30,7 +30,7 @@
 // with every float32 operand as its (hi, lo) pair (hi hi + hi lo + lo hi; v is a bfloat16 projection,
 // one term), so nothing that enters the recurrence is rounded below 2^-16; decays are applied to
 // float32 values.
-#include "sigmoid_attention_mma.cuh"      // ldmatrix / mma.sync / cp.async helpers
+#include "linear_chunks.cuh"
 
 namespace {
 
@@ -39,6 +39,7 @@ using sa_mma::ldsm_x4;
 using sa_mma::ldsm_x4_trans;
 using sa_mma::mma_bf16;
 using sa_mma::pack_bf16;
+using namespace chunks;
 
 // one element of a q or k head behind the rotation; `get(d)` gives the head's projected elements
 template <typename Get>
@@ -59,19 +60,6 @@ __device__ __forceinline__ float turned(Get get, int d, int rot, float pos, cons
 // while the sequence's tokens are walked (else in the slot; a sequence on slot 0 then forgets
 // each token).
 constexpr int ST = 256;
-template <int VEC> struct Cols;
-template <> struct Cols<4> { using T = float4; };
-template <> struct Cols<1> { using T = float; };
-__device__ __forceinline__ void col_step(float4& s, float4& o, float d, float k, float q, const float4& v) {
-  s.x = __fmaf_rn(k, v.x, __fmul_rn(d, s.x)); o.x = __fmaf_rn(s.x, q, o.x);
-  s.y = __fmaf_rn(k, v.y, __fmul_rn(d, s.y)); o.y = __fmaf_rn(s.y, q, o.y);
-  s.z = __fmaf_rn(k, v.z, __fmul_rn(d, s.z)); o.z = __fmaf_rn(s.z, q, o.z);
-  s.w = __fmaf_rn(k, v.w, __fmul_rn(d, s.w)); o.w = __fmaf_rn(s.w, q, o.w);
-}
-__device__ __forceinline__ void col_step(float& s, float& o, float d, float k, float q, const float& v) {
-  s = __fmaf_rn(k, v, __fmul_rn(d, s));
-  o = __fmaf_rn(s, q, o);
-}
 
 template <int VEC>
 __global__ void __launch_bounds__(ST)
@@ -170,33 +158,6 @@ retention_step_kernel(Source proj, long long row_width, const float* __restrict_
 }
 
 // ---- chunks ----------------------------------------------------------------------------------------
-constexpr int CH = 64;        // tokens of a chunk
-constexpr int PAD = 8;        // bfloat16 elements of padding per shared-memory row
-
-// Chunk c of sequence b (of the B whose boundaries `cu` gives) has the place (cu[b] - cu[0]) / CH + b + c:
-// no two chunks share one, and no list is needed.  Returns false for a place without a chunk.
-__device__ __forceinline__ int first_place(const int* cu, int b) { return (cu[b] - cu[0]) / CH + b; }
-__device__ __forceinline__ bool chunk_at(const int* cu, int B, int place, int& b, int& first, int& count) {
-  int lo = 0, hi = B - 1;
-  while (lo < hi) {             // the last sequence whose first place is not behind this one
-    const int mid = (lo + hi + 1) >> 1;
-    if (first_place(cu, mid) <= place) lo = mid;
-    else hi = mid - 1;
-  }
-  b = lo;
-  const int len = cu[b + 1] - cu[b];
-  first = (place - first_place(cu, b)) * CH;
-  count = len - first < CH ? len - first : CH;
-  return count > 0;
-}
-
-__device__ __forceinline__ void split2(float x, float y, unsigned& hi, unsigned& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  hi = *reinterpret_cast<const unsigned*>(&h);
-  const float2 f = __bfloat1622float2(h);
-  lo = pack_bf16(__fsub_rn(x, f.x), __fsub_rn(y, f.y));
-}
-
 // planes: qh, ql, kh, kl, each [tokens][H N] (plane elements apart)
 __global__ void __launch_bounds__(256)
 retention_rotate_kernel(const __nv_bfloat16* proj, long long row_width, const float* __restrict__ freq, int rot,
@@ -578,8 +539,6 @@ retention_output_kernel(const __nv_bfloat16* planes, long long plane, const __nv
     }
   }
 }
-
-constexpr int MOST_SMEM = 224 * 1024;
 
 template <int NPT, int OUT_NPT, int HALVES>
 int launch_chunks(const __nv_bfloat16* planes, long long plane, const __nv_bfloat16* proj, long long row_width,

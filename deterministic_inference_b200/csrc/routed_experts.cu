@@ -1,7 +1,9 @@
 // A feed-forward of routed experts: the router's choice, the sort of (token, expert) pairs into
 // tiles of one expert each, the two grouped products, and the weighted sum.
 //
-//   route:    s = sigmoid(z), or softmax(z) over all experts (score_kind 1); choice = s + correction;
+//   route:    s = sigmoid(z), or softmax(z) over all experts (score_kind 1); choice = s + correction (which
+//             may be absent); or (score_kind 2) choice = z (+ correction) and s = exp(z - largest z), whose
+//             share of the chosen ones' sum is the softmax over the chosen logits alone;
 //             experts in equal groups of neighbours, a group's score the sum of its `group_top` (1 or
 //             2) largest choice scores, the best `group_keep` groups stay; of their experts the `top`
 //             largest choice scores win (ties: the lower index); weight_j = s_j / (sum of the chosen
@@ -11,7 +13,8 @@
 //   sort:     pairs p = t * top + j are placed, by expert, into tiles of `tile` rows; an expert's
 //             rows are filled up to whole tiles (row -> pair or -1; tile -> expert or -1).
 //   gate/up:  hidden[row] = act(x[token] Wg_e^T, x[token] Wu_e^T), rounded once to x's type; act(g, u) =
-//             silu(g) u, or, limited, min(g, l) sigmoid(alpha min(g, l)) (clamp(u, -l, l) + 1).
+//             silu(g) u, or, limited, min(g, l) sigmoid(alpha min(g, l)) (clamp(u, -l, l) + 1).  Experts
+//             without a gate: hidden[row] = z (1 + erf(z / sqrt 2)) / 2 with z = x[token] Wu_e^T.
 //   down:     per_pair[pair] = hidden[row] Wd_e^T, float32.
 //   combine:  out[t] = sum_j weight[t, j] (or the constant) per_pair[t * top + j] (in the order of j)
 //                      + sigmoid(logits[t, col]) * shared[t] (col < 0: + shared[t]).
@@ -53,7 +56,19 @@ moe_route_kernel(Source logits, long long row_width, const float* __restrict__ c
   float* choice = s + E;
   float* gscore = choice + E;
   const int per = E / groups;
-  if (score_kind == 1) {
+  if (score_kind == 2) {
+    float mx = NEG_INF;
+    for (int e = lane; e < E; e += 32) {
+      const float z = source_load(logits, (long long)t * row_width + e);
+      s[e] = z;
+      mx = fmaxf(mx, z);
+    }
+    mx = warp_max(mx);
+    for (int e = lane; e < E; e += 32) {
+      choice[e] = correction != nullptr ? __fadd_rn(s[e], correction[e]) : s[e];
+      s[e] = expf(s[e] - mx);
+    }
+  } else if (score_kind == 1) {
     // softmax over all experts: the largest logit, then the sum of the exponentials in a fixed order
     float mx = NEG_INF;
     for (int e = lane; e < E; e += 32) {
@@ -72,13 +87,13 @@ moe_route_kernel(Source logits, long long row_width, const float* __restrict__ c
     for (int e = lane; e < E; e += 32) {
       const float v = s[e] / den;
       s[e] = v;
-      choice[e] = __fadd_rn(v, correction[e]);
+      choice[e] = correction != nullptr ? __fadd_rn(v, correction[e]) : v;
     }
   } else {
     for (int e = lane; e < E; e += 32) {
       const float v = sigmoid_f32(source_load(logits, (long long)t * row_width + e));
       s[e] = v;
-      choice[e] = __fadd_rn(v, correction[e]);
+      choice[e] = correction != nullptr ? __fadd_rn(v, correction[e]) : v;
     }
   }
   __syncwarp();
@@ -191,6 +206,7 @@ moe_sort_kernel(const int* ids, const int* __restrict__ table, int top, int V, i
 // mode 0 (gate and up): A row r = x[pair / top] (K = the model's width), B = the expert's [2F][K] (gate
 // rows, then up rows), out hidden[row][F] = act(gate, up) in T.
 // mode 1 (down): A row r = hidden[row] (K = F), B = the expert's [N][K], out per_pair[pair][N] float32.
+// mode 2 (up alone): A as in mode 0, B as in mode 1, out hidden[row][N] = the erf gelu of the product in T.
 
 // limit > 0: the limited gate; else silu
 __device__ __forceinline__ float expert_gate(float g, float u, float limit, float alpha) {
@@ -201,6 +217,8 @@ __device__ __forceinline__ float expert_gate(float g, float u, float limit, floa
   }
   return g * sigmoid_f32(g) * u;
 }
+
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
 
 __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3,
                                                unsigned b0, unsigned b1) {
@@ -262,7 +280,7 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ a_rows, const int* __re
       const int pair = row_pair[r];
       uint4 v = make_uint4(0, 0, 0, 0);
       if (pair >= 0 && c8 * 8 < klen) {
-        const long long arow = mode == 0 ? pair / top : (long long)tl * tile + r;
+        const long long arow = mode != 1 ? pair / top : (long long)tl * tile + r;
         v = *reinterpret_cast<const uint4*>(a_rows + arow * K + kc + c8 * 8);
       }
       *reinterpret_cast<uint4*>(As + r * as + c8 * 8) = v;
@@ -315,6 +333,15 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ a_rows, const int* __re
             const float gt = acc[m][j][2 * hh + e], up = acc[m][j + HALF][2 * hh + e];
             if (n < N) dst[n] = __float2bfloat16_rn(expert_gate(gt, up, limit, alpha));
           }
+      } else if (mode == 2) {
+        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + ((long long)tl * tile + r) * N;
+#pragma unroll
+        for (int j = 0; j < NJ; ++j)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int n = n0 + j * 8 + tig * 2 + e;
+            if (n < N) dst[n] = __float2bfloat16_rn(gelu_erf(acc[m][j][2 * hh + e]));
+          }
       } else {
         float* dst = reinterpret_cast<float*>(out) + (long long)pair * N;
 #pragma unroll
@@ -360,7 +387,7 @@ moe_product_kernel(const T* __restrict__ a_rows, const int* __restrict__ order, 
       const int pair = row_pair[r];
       float v = 0.f;
       if (pair >= 0 && k < klen) {
-        const long long arow = mode == 0 ? pair / top : (long long)tl * tile + r0 + r;
+        const long long arow = mode != 1 ? pair / top : (long long)tl * tile + r0 + r;
         v = Elem<T>::load(a_rows + arow * K + kc + k);
       }
       xs[r][k] = v;
@@ -385,6 +412,8 @@ moe_product_kernel(const T* __restrict__ a_rows, const int* __restrict__ order, 
     if (mode == 0)
       Elem<T>::store(reinterpret_cast<T*>(out) + ((long long)tl * tile + r0 + r) * N + n,
                      expert_gate(acc0[r], acc1[r], limit, alpha));
+    else if (mode == 2)
+      Elem<T>::store(reinterpret_cast<T*>(out) + ((long long)tl * tile + r0 + r) * N + n, gelu_erf(acc0[r]));
     else
       reinterpret_cast<float*>(out)[(long long)pair * N + n] = acc0[r];
   }
@@ -431,7 +460,7 @@ int launch_product_mma(const void* a_rows, const int* order, int max_tiles, int 
   return DIB_OK;
 }
 
-// mode 0: gate and up; 1: down.  dtype 0 float32, 1 bfloat16.
+// mode 0: gate and up; 1: down; 2: up alone.  dtype 0 float32, 1 bfloat16.
 int moe_product(const void* a_rows, int dtype, const int* order, int max_tiles, int tile, int top, const void* w,
                 void* out, int K, int N, int mode, float limit, float alpha, cudaStream_t st) {
   if (max_tiles == 0) return DIB_OK;
@@ -512,7 +541,7 @@ int dib_moe_route(const void* logits, int kind, int splits, long long stride, lo
                   float scale, float eps, int score_kind, int group_top, int normalize, cudaStream_t st) {
   if (T == 0) return DIB_OK;
   if (E < 1 || E > 1024 || top < 1 || top > 32 || groups < 1 || E % groups || keep < 1 || keep > groups ||
-      top > keep * (E / groups) || score_kind < 0 || score_kind > 1 || group_top < 1 || group_top > 2)
+      top > keep * (E / groups) || score_kind < 0 || score_kind > 2 || group_top < 1 || group_top > 2)
     return DIB_BAD_SIZE;
   const size_t smem = sizeof(float) * ROUTE_WARPS * (2 * (size_t)E + groups);
   dib_launch(moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, st,
@@ -537,6 +566,12 @@ int dib_moe_sort(const int* ids, const int* table, int top, int V, int pairs, in
 int dib_moe_gate_up(const void* x, int dtype, const int* order, int max_tiles, int tile, int top, const void* w_gate_up,
                     void* hidden, int F, int W, float limit, float alpha, cudaStream_t st) {
   return moe_product(x, dtype, order, max_tiles, tile, top, w_gate_up, hidden, W, F, 0, limit, alpha, st);
+}
+
+// experts without a gate: w_up [experts][F][W], hidden = the erf gelu of the product
+int dib_moe_up(const void* x, int dtype, const int* order, int max_tiles, int tile, int top, const void* w_up, void* hidden,
+               int F, int W, cudaStream_t st) {
+  return moe_product(x, dtype, order, max_tiles, tile, top, w_up, hidden, W, F, 2, 0.f, 0.f, st);
 }
 
 int dib_moe_down(const void* hidden, int dtype, const int* order, int max_tiles, int tile, const void* w_down,

@@ -1,6 +1,6 @@
 // Kernels of models whose residual stream is kept in float32 whatever the engine's
-// storage type is: token + learned position embedding, RMSNorm of the float32 stream
-// (alone, or after adding up to two scaled mixer outputs to it), the scaled sum as a
+// storage type is: token + learned position embedding, RMSNorm or layer norm of the float32 stream
+// (alone, or after adding up to three scaled outputs to it), the scaled sum as a
 // tensor, the xIELU activation and the soft cap of the logits.  All arithmetic is float32;
 // inputs that come from a matrix product may be its split-k partial products.
 #include "source.cuh"
@@ -241,6 +241,151 @@ __global__ void stream_norm_normed_terms_kernel(float* residual, int terms, Sour
     store_as(out, out_dtype, base + c, residual[base + c] * rstd * w[c]);
 }
 
+// One block per row: stream[row] += sum_k a_k * n_k(x_k[row] + bias_k), the terms' sum taken first (in
+// their order) and then added, nothing rounded below float32; n_k(v) = v / sqrt(mean(v^2) + e_k) * w_k
+// where the term has a weight, v where it has none.  Then, when out is given, out[row] = the stream
+// itself (norm_kind 0), its RMS norm stream / sqrt(mean(stream^2) + eps) * w (1), or its layer norm
+// (stream - mean) / sqrt(mean((stream - mean)^2) + eps) * w (2).
+// The block's width depends on W alone, and a sum over a row is a thread's own elements in ascending order,
+// then the block's; VPT > 0 keeps a thread's elements in registers, VPT 0 reads them again.
+struct StreamTerm {
+  Source x;
+  float a;
+  const float* bias;
+  const float* w;
+  float eps;
+};
+constexpr int STREAM_TERMS = 3;
+struct StreamTerms {
+  StreamTerm t[STREAM_TERMS];
+  int n;
+};
+
+template <int VPT, int AHEAD>
+__global__ void stream_terms_kernel(float* stream, StreamTerms terms, int norm_kind, const float* w, void* out,
+                                    int out_dtype, int W, float eps) {
+  __shared__ float scratch[32];
+  pdl_prologue(stream, terms.t[0].x.p, terms.t[1].x.p, terms.t[2].x.p);
+  const long long base = (long long)blockIdx.x * W;
+  const float width = (float)W;
+  if (VPT > 0) {
+    constexpr int N = VPT > 0 ? VPT : 1;
+    float r[N], sum[N], v[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      r[i] = c < W ? stream[base + c] : 0.f;
+      sum[i] = 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < STREAM_TERMS; ++k) {
+      if (k >= terms.n) break;
+      const StreamTerm& t = terms.t[k];
+      source_load_strided<N, AHEAD>(t.x, base, threadIdx.x, blockDim.x, W, v);
+      if (t.bias != nullptr) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+          const int c = threadIdx.x + i * blockDim.x;
+          if (c < W) v[i] = __fadd_rn(v[i], t.bias[c]);
+        }
+      }
+      if (t.w != nullptr) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < N; ++i) ss = __fmaf_rn(v[i], v[i], ss);
+        const float f = 1.0f / sqrtf(block_sum(ss, scratch) / width + t.eps);
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+          const int c = threadIdx.x + i * blockDim.x;
+          if (c < W) v[i] = __fmul_rn(__fmul_rn(v[i], f), t.w[c]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < N; ++i) sum[i] = __fmaf_rn(t.a, v[i], sum[i]);
+    }
+    float first = 0.f;                      // the row's sum (layer norm) or its squares' (RMS norm)
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < W) {
+        if (terms.n > 0) {
+          r[i] = __fadd_rn(r[i], sum[i]);
+          stream[base + c] = r[i];
+        }
+        first = norm_kind == 2 ? __fadd_rn(first, r[i]) : __fmaf_rn(r[i], r[i], first);
+      }
+    }
+    if (out == nullptr) return;
+    float mean = 0.f, rstd = 1.f;
+    if (norm_kind == 1) rstd = 1.0f / sqrtf(block_sum(first, scratch) / width + eps);
+    if (norm_kind == 2) {
+      mean = block_sum(first, scratch) / width;
+      float sq = 0.f;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < W) {
+          const float d = __fsub_rn(r[i], mean);
+          sq = __fmaf_rn(d, d, sq);
+        }
+      }
+      rstd = 1.0f / sqrtf(block_sum(sq, scratch) / width + eps);
+    }
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < W) store_as(out, out_dtype, base + c, norm_kind == 0 ? r[i] : __fsub_rn(r[i], mean) * rstd * w[c]);
+    }
+    return;
+  }
+  float f[STREAM_TERMS];
+#pragma unroll
+  for (int k = 0; k < STREAM_TERMS; ++k) {
+    f[k] = 1.f;
+    if (k >= terms.n || terms.t[k].w == nullptr) continue;
+    const StreamTerm& t = terms.t[k];
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+      float v = source_load(t.x, base + c);
+      if (t.bias != nullptr) v = __fadd_rn(v, t.bias[c]);
+      ss = __fmaf_rn(v, v, ss);
+    }
+    f[k] = 1.0f / sqrtf(block_sum(ss, scratch) / width + t.eps);
+  }
+  float first = 0.f;
+  for (int c = threadIdx.x; c < W; c += blockDim.x) {
+    float r = stream[base + c], sum = 0.f;
+#pragma unroll
+    for (int k = 0; k < STREAM_TERMS; ++k) {
+      if (k >= terms.n) break;
+      const StreamTerm& t = terms.t[k];
+      float v = source_load(t.x, base + c);
+      if (t.bias != nullptr) v = __fadd_rn(v, t.bias[c]);
+      if (t.w != nullptr) v = __fmul_rn(__fmul_rn(v, f[k]), t.w[c]);
+      sum = __fmaf_rn(t.a, v, sum);
+    }
+    if (terms.n > 0) {
+      r = __fadd_rn(r, sum);
+      stream[base + c] = r;
+    }
+    first = norm_kind == 2 ? __fadd_rn(first, r) : __fmaf_rn(r, r, first);
+  }
+  if (out == nullptr) return;
+  float mean = 0.f, rstd = 1.f;
+  if (norm_kind == 1) rstd = 1.0f / sqrtf(block_sum(first, scratch) / width + eps);
+  if (norm_kind == 2) {
+    mean = block_sum(first, scratch) / width;
+    float sq = 0.f;
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+      const float d = __fsub_rn(stream[base + c], mean);
+      sq = __fmaf_rn(d, d, sq);
+    }
+    rstd = 1.0f / sqrtf(block_sum(sq, scratch) / width + eps);
+  }
+  for (int c = threadIdx.x; c < W; c += blockDim.x)
+    store_as(out, out_dtype, base + c, norm_kind == 0 ? stream[base + c] : __fsub_rn(stream[base + c], mean) * rstd * w[c]);
+}
+
 // out = a0 * x0 (+ a1 * x1), float32
 __global__ void weighted_sum_kernel(Source x0, float a0, Source x1, float a1, int terms, float* out,
                                     long long n) {
@@ -396,6 +541,36 @@ int dib_stream_norm_normed_terms(float* residual, int terms, const void* x0, int
   const dim3 grid(rows), block(W >= 2048 ? 512 : (W >= 512 ? 256 : 128));
   dib_launch(stream_norm_normed_terms_kernel, grid, block, 0, st, residual, terms, s0, a0, w0, e0, s1, a1, w1, e1, w,
              out, out_dtype, W, eps);
+  DIB_CHECK_LAUNCH();
+  return DIB_OK;
+}
+
+// Up to three terms (see stream_terms_kernel).  x null with terms == 0.  out null: the stream is updated
+// only.  norm_kind 0: out is the stream in out's type; 1: its RMS norm; 2: its layer norm.
+int dib_stream_terms(float* stream, int terms, const void* x0, int kind0, int splits0, long long stride0, float a0,
+                     const float* b0, const float* w0, float e0, const void* x1, int kind1, int splits1,
+                     long long stride1, float a1, const float* b1, const float* w1, float e1, const void* x2, int kind2,
+                     int splits2, long long stride2, float a2, const float* b2, const float* w2, float e2, int norm_kind,
+                     const float* w, void* out, int out_dtype, int rows, int W, float eps, cudaStream_t st) {
+  if (rows == 0) return DIB_OK;
+  if (W < 1 || terms < 0 || terms > STREAM_TERMS || norm_kind < 0 || norm_kind > 2) return DIB_BAD_SIZE;
+  if (out != nullptr && ((norm_kind > 0 && w == nullptr) || (out_dtype != 0 && out_dtype != 1))) return DIB_BAD_DTYPE;
+  StreamTerms t;
+  t.n = terms;
+  t.t[0] = {make_source(x0, kind0, splits0, stride0), a0, b0, w0, e0};
+  t.t[1] = {make_source(x1, kind1, splits1, stride1), a1, b1, w1, e1};
+  t.t[2] = {make_source(x2, kind2, splits2, stride2), a2, b2, w2, e2};
+  bool split = false;
+  for (int k = 0; k < terms; ++k) split = split || t.t[k].x.splits > 1;
+  const dim3 grid(rows), block(W >= 2048 ? 512 : (W >= 512 ? 256 : 128));
+  const int per_thread = (W + (int)block.x - 1) / (int)block.x;
+#define DIB_ST(VPT, AHEAD) dib_launch(stream_terms_kernel<VPT, AHEAD>, grid, block, 0, st, stream, t, norm_kind, w, out, out_dtype, W, eps)
+  if (per_thread <= 4 && split) DIB_ST(4, 4);
+  else if (per_thread <= 4) DIB_ST(4, 0);
+  else if (per_thread <= 8 && split) DIB_ST(8, 2);
+  else if (per_thread <= 8) DIB_ST(8, 0);
+  else DIB_ST(0, 0);
+#undef DIB_ST
   DIB_CHECK_LAUNCH();
   return DIB_OK;
 }

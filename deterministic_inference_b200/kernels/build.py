@@ -48,6 +48,7 @@ SOURCES = {
     "routed_experts": "routed_experts.cu",
     "state_space": "state_space.cu",
     "retention": "retention.cu",
+    "gated_linear_attention": "gated_linear_attention.cu",
 }
 HEADERS = ("common.cuh", "attention_merge.cuh")
 # further headers a library includes
@@ -62,7 +63,8 @@ EXTRA_HEADERS = {
     "state_space": ("source.cuh", "conv_tail.cuh"),
     "linear_recurrence": ("source.cuh", "conv_tail.cuh"),
     "routed_experts": ("source.cuh",),
-    "retention": ("source.cuh", "sigmoid_attention_mma.cuh"),
+    "retention": ("source.cuh", "sigmoid_attention_mma.cuh", "linear_chunks.cuh"),
+    "gated_linear_attention": ("source.cuh", "sigmoid_attention_mma.cuh", "linear_chunks.cuh"),
 }
 
 NVCC_FLAGS = [

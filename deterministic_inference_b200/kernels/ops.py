@@ -260,14 +260,14 @@ class SplitAttention:
 
 class WeightedSum:
     """sum_i scale_i * term_i that is not computed yet: the outputs of mixers that run side
-    by side, each a tensor, a ``SplitSum`` or a ``NormedTerm`` (an output that is RMS-normed
+    by side, each a tensor, a ``SplitSum``, a ``BiasedTerm`` or a ``NormedTerm`` (an output that is RMS-normed
     with a weight of its own before it is scaled).  The norm of a float32 residual stream adds
     the terms to the stream in their order while it loads them; ``tensor()`` gives the sum
     as a float32 tensor."""
 
     def __init__(self, terms: list):
-        if not 1 <= len(terms) <= 2:
-            raise KernelError(f"a weighted sum of {len(terms)} terms has no kernel (1 or 2)")
+        if not 1 <= len(terms) <= STREAM_TERMS:
+            raise KernelError(f"a weighted sum of {len(terms)} terms has no kernel (1 to {STREAM_TERMS})")
         self.terms = [(float(a), x) for a, x in terms]
         self.dtype = torch.float32
 
@@ -285,6 +285,9 @@ class WeightedSum:
 
     def tensor(self) -> torch.Tensor:
         rows, width = self.shape
+        if needs_stream_terms(self):
+            out = torch.zeros(rows, width, dtype=torch.float32, device=self.device)
+            return stream_terms_(out, self)
         if self.normed:
             out = torch.zeros(rows, width, dtype=torch.float32, device=self.device)
             _stream_add_normed_terms(out, self.terms, None, 0.0, None)
@@ -320,7 +323,93 @@ class NormedTerm:
         return stream_add_(out, self)
 
 
-_DEFERRED = (SplitSum, GatedSplit, SplitAttention, WeightedSum, NormedTerm)
+class BiasedTerm:
+    """x + bias that is not computed yet: a projection (a tensor or a ``SplitSum``) whose bias (a float32
+    vector) the float32 residual stream adds while it loads the rows, before anything is rounded or normed;
+    ``tensor()`` gives it as a float32 tensor."""
+
+    def __init__(self, x, bias: torch.Tensor):
+        self.x, self.bias = x, bias
+        self.dtype = torch.float32
+
+    @property
+    def shape(self):
+        return self.x.shape
+
+    @property
+    def device(self):
+        return self.x.device
+
+    def tensor(self) -> torch.Tensor:
+        rows, width = self.shape
+        out = torch.zeros(rows, width, dtype=torch.float32, device=self.device)
+        return stream_terms_(out, self)
+
+
+# most terms a float32 residual stream takes in one kernel
+STREAM_TERMS = 3
+
+
+def needs_stream_terms(x) -> bool:
+    """Whether a pending term is one that only ``stream_terms_`` adds to a stream: a bias, or more than two
+    terms."""
+    if isinstance(x, WeightedSum):
+        return len(x.terms) > 2 or any(needs_stream_terms(t) for _, t in x.terms)
+    return isinstance(x, BiasedTerm) or (isinstance(x, NormedTerm) and isinstance(x.x, BiasedTerm))
+
+
+STREAM_NORMS = {None: 0, "rms": 1, "layer": 2}
+
+
+def stream_terms_(stream: torch.Tensor, term=None, norm=None, weight=None, eps: float = 0.0, out=None) -> torch.Tensor:
+    """In place, float32: stream += term (a tensor, a ``SplitSum``, a ``BiasedTerm``, a ``NormedTerm`` of those, or a
+    ``WeightedSum`` of up to STREAM_TERMS; their sum is taken first and nothing is rounded on the way).  With
+    ``out`` also out = the stream in out's type (``norm`` None), its RMS norm ("rms") or its layer norm
+    ("layer": (x - mean) / sqrt(mean((x - mean)^2) + eps)), times ``weight``.  Returns the stream."""
+    _need(stream, "stream", torch.float32, 2)
+    rows, w = stream.shape
+    terms = [] if term is None else term.terms if isinstance(term, WeightedSum) else [(1.0, term)]
+    if norm not in STREAM_NORMS or len(terms) > STREAM_TERMS:
+        raise KernelError(f"stream_terms_: norm {norm!r} ({list(STREAM_NORMS)}), {len(terms)} terms (at most {STREAM_TERMS})")
+    args = []
+    for a, x in terms:
+        if tuple(x.shape) != (rows, w):
+            raise KernelError(f"stream_terms_: a term of shape {tuple(x.shape)} for a stream {(rows, w)}")
+        wx, ex, bias = None, 0.0, None
+        if isinstance(x, NormedTerm):
+            wx, ex, x = x.weight, x.eps, x.x
+        if isinstance(x, BiasedTerm):
+            bias, x = x.bias, x.x
+        for v, name in ((wx, "a term's norm weight"), (bias, "a term's bias")):
+            if v is not None:
+                _need(v, name, torch.float32, 1)
+                if v.shape[0] != w:
+                    raise KernelError(f"stream_terms_: {name} has {v.shape[0]} elements, rows have {w}")
+        args += [*_source_args(x), c_float(a), _ptr(bias), _ptr(wx), c_float(ex)]
+    for _ in range(STREAM_TERMS - len(terms)):
+        args += [c_void_p(0), c_int(0), c_int(1), c_longlong(0), c_float(0.0), c_void_p(0), c_void_p(0), c_float(0.0)]
+    if out is not None:
+        _need(out, "out", None, 2)
+        if norm is not None:
+            _need(weight, "weight", torch.float32, 1)
+            if weight.shape[0] != w:
+                raise KernelError(f"stream_terms_: weight has {weight.shape[0]} elements, rows have {w}")
+    st = _lib("stream_f32").dib_stream_terms(
+        _ptr(stream), c_int(len(terms)), *args, c_int(STREAM_NORMS[norm]), _ptr(weight), _ptr(out),
+        c_int(_DT[out.dtype] if out is not None else 0), c_int(rows), c_int(w), c_float(eps), _stream())
+    _check(st, "stream_terms_", f"row width {w}")
+    return stream
+
+
+def stream_layer_norm(stream: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype, add=None) -> torch.Tensor:
+    """Layer norm (a weight, no bias) of the float32 residual stream, written in ``out_dtype``; with ``add``
+    (any pending term) the stream first takes stream += add in place, in float32."""
+    out = torch.empty(stream.shape, dtype=out_dtype, device=stream.device)
+    stream_terms_(stream, add, "layer", weight, eps, out)
+    return out
+
+
+_DEFERRED = (SplitSum, GatedSplit, SplitAttention, WeightedSum, NormedTerm, BiasedTerm)
 
 
 def _source_args(x):
@@ -628,6 +717,8 @@ def gather_rows(x: torch.Tensor, index: torch.Tensor) -> torch.Tensor:
     """out[r] = x[index[r]]; index int32."""
     if isinstance(x, NormedTerm):          # a norm works row by row: gather first
         return NormedTerm(gather_rows(x.x, index), x.weight, x.eps)
+    if isinstance(x, BiasedTerm):
+        return BiasedTerm(gather_rows(x.x, index), x.bias)
     if isinstance(x, WeightedSum):
         return WeightedSum([(a, gather_rows(term, index)) for a, term in x.terms])
     x = as_tensor(x)
@@ -803,6 +894,10 @@ def stream_rms_norm(stream: torch.Tensor, weight: torch.Tensor, eps: float, out_
     rows, w = stream.shape
     if weight.shape[0] != w:
         raise KernelError(f"stream_rms_norm: weight has {weight.shape[0]} elements, rows have {w}")
+    if needs_stream_terms(add):
+        out = torch.empty(rows, w, dtype=out_dtype, device=stream.device)
+        stream_terms_(stream, add, "rms", weight, eps, out)
+        return out
     if isinstance(add, NormedTerm):
         out = torch.empty(rows, w, dtype=out_dtype, device=stream.device)
         stream_add_(stream, add, norm_weight=weight, norm_eps=eps, out=out)
@@ -855,15 +950,18 @@ def stream_add_(stream: torch.Tensor, term=None, bias=None, norm_weight=None, no
 
 
 def stream_read(stream: torch.Tensor, term, out_dtype) -> torch.Tensor:
-    """The float32 residual stream as the next sublayer reads it: first stream += term in place (a
-    ``NormedTerm`` computed in float32 and never rounded, or None), then the stream itself in
-    ``out_dtype`` (float32: the stream, no copy)."""
+    """The float32 residual stream as the next sublayer reads it: first stream += term in place (any pending
+    term, never rounded below float32, or None), then the stream itself in ``out_dtype`` (float32: the
+    stream, no copy)."""
     _need(stream, "stream", torch.float32, 2)
-    if out_dtype == torch.float32:
-        return stream if term is None else stream_add_(stream, term)
-    out = torch.empty(stream.shape, dtype=out_dtype, device=stream.device)
-    stream_add_(stream, term, out=out)
-    return out
+    out = None if out_dtype == torch.float32 else torch.empty(stream.shape, dtype=out_dtype, device=stream.device)
+    if term is None and out is None:
+        return stream
+    if term is None or (isinstance(term, NormedTerm) and not needs_stream_terms(term)):
+        stream_add_(stream, term, out=out)
+    else:
+        stream_terms_(stream, term, out=out)
+    return stream if out is None else out
 
 
 def embedding_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float) -> torch.Tensor:
@@ -1314,6 +1412,80 @@ def retention(proj, decay: torch.Tensor, freq, state: torch.Tensor, step, num_he
     return out
 
 
+# ---------------------------------------------------------------- gated linear attention
+
+# DIB200_GLA_CHUNKED=0 (read once): prompt portions run token by token too
+GLA_CHUNKED = __import__("os").environ.get("DIB200_GLA_CHUNKED", "1") != "0"
+
+
+def gated_linear_attention(proj, hidden, hidden_col: int, a2_t: torch.Tensor, a2_bias: torch.Tensor, tau: float,
+                           norm_weight: torch.Tensor, state: torch.Tensor, step, num_heads: int, head_dim: int,
+                           v_head_dim: int, norm_eps: float, out_dtype) -> torch.Tensor:
+    """Gated linear attention over every sequence's tokens of the step: [T, H * E] in ``out_dtype``.  ``proj``
+    rows are [q: H D | k: H D | v: H E | g: H E | anything]; ``hidden`` rows hold, from column ``hidden_col`` on,
+    the R inputs of the decay map (float32 sums): alpha = sigmoid(z)^(1/tau) with z = hidden a2_t + a2_bias
+    (``a2_t`` [R, H D]).  Per head S <- diag(alpha) S + k v^T, o = S^T (q D^(-1/2)), from and to ``state`` float32
+    [slots, H D E] (rows ``step.state_slots``); then each head's o over its root mean square (``norm_eps``), times
+    ``norm_weight`` [E], times silu(g).  The step's leading one-token sequences, and every sequence of the float32
+    engine or of sizes the chunked form does not take, run token by token; other portions in chunks on the tensor
+    cores, so which form a sequence runs on depends on what IT brings."""
+    t, width = proj.shape
+    h, d, e = num_heads, head_dim, v_head_dim
+    if width < 2 * h * (d + e):
+        raise KernelError(f"gated_linear_attention: projection rows of {width}, expected at least {2 * h * (d + e)}")
+    _need(a2_t, "a2_t", None, 2)
+    _need(a2_bias, "a2_bias", torch.float32, 1)
+    _need(norm_weight, "norm_weight", torch.float32, 1)
+    _need(state, "state", torch.float32, 2)
+    rank = a2_t.shape[0]
+    if a2_t.shape[1] != h * d or a2_bias.shape[0] != h * d or norm_weight.shape[0] != e or state.shape[1] != h * d * e \
+            or hidden.shape[0] != t or hidden.shape[1] < hidden_col + rank or not tau > 0:
+        raise KernelError(f"gated_linear_attention: a weight, the decay map's input or the state does not fit {h} heads "
+                          f"of {d}/{e}")
+    lib = _lib("gated_linear_attention")
+    dev = state.device
+    log_decay = torch.empty(t, h * d, dtype=torch.float32, device=dev)
+    st = lib.dib_gla_decay(*_source_args(hidden), c_longlong(hidden.shape[1]), c_longlong(hidden_col), _ptr(a2_t),
+                           c_int(_dt(a2_t, "a2_t")), _ptr(a2_bias), c_float(tau), _ptr(log_decay), c_int(t), c_int(rank),
+                           c_int(h * d), _stream())
+    _check(st, "gated_linear_attention(decays)", f"a map of rank {rank} (at most 1024)")
+    out = torch.empty(t, h * e, dtype=out_dtype, device=dev)
+    n, nd = step.num_seqs, min(int(step.num_decode or 0), step.num_seqs)
+    chunked = GLA_CHUNKED and out_dtype == torch.bfloat16 and d % 16 == 0 and e % 16 == 0 and d <= 256 and e <= 256 \
+        and width % 8 == 0
+    q_scale = float(d) ** -0.5
+    stride = c_longlong(state.shape[1])
+
+    def by_token(first, count, in_smem):
+        st = lib.dib_gla_step(*_source_args(proj), c_longlong(width), _ptr(log_decay), _ptr(state), stride,
+                              c_void_p(step.cu_q_lens.data_ptr() + 4 * first),
+                              c_void_p(step.state_slots.data_ptr() + 4 * first), _ptr(norm_weight), _ptr(out),
+                              c_int(_DT[out_dtype]), c_int(count), c_int(h), c_int(d), c_int(e), c_float(q_scale),
+                              c_float(norm_eps), c_int(in_smem), _stream())
+        _check(st, "gated_linear_attention(token by token)", f"heads of {d}/{e}")
+
+    if nd:
+        by_token(0, nd, 0)
+    if nd < n and not chunked:
+        by_token(nd, n - nd, int(lib.dib_gla_state_fits(c_int(d), c_int(e))))
+    elif nd < n:
+        if isinstance(proj, SplitSum) or proj.dtype != torch.bfloat16:      # the stored bfloat16 matrix
+            parts = proj.parts if isinstance(proj, SplitSum) else as_tensor(proj).unsqueeze(0)
+            proj = SplitSum(parts, torch.bfloat16).tensor()
+        tokens = t - nd
+        places = tokens // 64 + n - nd
+        planes = torch.empty(4, tokens, h * d, dtype=torch.bfloat16, device=dev)
+        edges = torch.empty(places, h, 8, d, dtype=torch.float32, device=dev)
+        sums = torch.empty(places, h, d, e, dtype=torch.float32, device=dev)
+        st = lib.dib_gla_chunked(_ptr(proj), c_longlong(width), _ptr(log_decay), _ptr(state), stride,
+                                 c_void_p(step.cu_q_lens.data_ptr() + 4 * nd),
+                                 c_void_p(step.state_slots.data_ptr() + 4 * nd), _ptr(norm_weight), _ptr(planes),
+                                 _ptr(edges), _ptr(sums), _ptr(out), c_int(n - nd), c_int(nd), c_int(tokens), c_int(h),
+                                 c_int(d), c_int(e), c_float(q_scale), c_float(norm_eps), _stream())
+        _check(st, "gated_linear_attention(chunks)", f"heads of {d}/{e}", kernels=4)
+    return out
+
+
 # ---------------------------------------------------------------- gated linear recurrent unit
 
 def gated_linear_recurrence(proj, bias: torch.Tensor, conv_weight: torch.Tensor, conv_bias: torch.Tensor,
@@ -1374,7 +1546,7 @@ EXPERT_TILE_ROWS_TC = 128
 EXPERTS_TC = __import__("os").environ.get("DIB200_EXPERTS_TC", "1") != "0"
 
 
-ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}
+ROUTER_SCORES = {"sigmoid": 0, "softmax": 1, "chosen_softmax": 2}
 
 
 def route_experts(logits, correction: torch.Tensor, num_experts: int, top: int, group_count: int,
@@ -1382,16 +1554,19 @@ def route_experts(logits, correction: torch.Tensor, num_experts: int, top: int, 
                   normalize: bool = True):
     """(int32 [T, top] chosen experts, float32 [T, top] their weights).  ``logits`` [T, >= E] (a float32
     tensor or split sums; columns from E on are not the router's): s = sigmoid(logits), or (``score``
-    "softmax") the softmax of the row's E logits; the choice is made on s + correction: the experts form
+    "softmax") the softmax of the row's E logits; the choice is made on s + correction (None: on s; ``score``
+    "chosen_softmax": the choice is made on the logits themselves, and the weights, with ``normalize``, are the
+    softmax over the chosen logits alone): the experts form
     ``group_count`` groups of neighbours, a group's score is the sum of its ``group_top`` (1 or 2)
     largest choice scores, the ``group_keep`` best groups stay, and of their experts the ``top`` largest
     choice scores win (ties: the lower index).  Weights: s of the chosen over their sum (+ eps), times
     ``scale``; with ``normalize`` off s times ``scale``."""
     t, row = logits.shape
-    _need(correction, "correction", torch.float32, 1)
+    if correction is not None:
+        _need(correction, "correction", torch.float32, 1)
     if score not in ROUTER_SCORES or group_top not in (1, 2):
         raise KernelError(f"route_experts: score {score!r} ({sorted(ROUTER_SCORES)}) or group_top {group_top} (1, 2)")
-    if correction.shape[0] != num_experts or row < num_experts or num_experts % group_count \
+    if (correction is not None and correction.shape[0] != num_experts) or row < num_experts or num_experts % group_count \
             or not 1 <= group_keep <= group_count or not 1 <= top <= group_keep * (num_experts // group_count):
         raise KernelError(f"route_experts: {num_experts} experts, rows of {row}, {group_count} groups, "
                           f"{group_keep} kept, {top} chosen")
@@ -1415,11 +1590,13 @@ class TableChoice:
 
 
 def routed_experts(x: torch.Tensor, ids, weights, w_gate_up: torch.Tensor,
-                   w_down: torch.Tensor, shared, logits, shared_gate_col: int, out_dtype, limited=None) -> torch.Tensor:
+                   w_down: torch.Tensor, shared, logits, shared_gate_col: int, out_dtype, limited=None,
+                   gated: bool = True) -> torch.Tensor:
     """float32 [T, W]: sum_j weights[t, j] * down_e(act(gate_e x_t, up_e x_t)) over the chosen experts
     e = ids[t, j], in the order of j (``ids`` a ``TableChoice``: the experts its table names, all with its
     weight; ``weights`` None).  act(g, u) = silu(g) u, or with ``limited`` = (limit, alpha) min(g, limit)
-    sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1).  Plus (``shared`` [T, W], a tensor or split sums, given)
+    sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1).  ``gated`` off: down_e(gelu(up_e x_t)) with the erf
+    gelu, and ``w_gate_up`` [E, F, W] holds the up rows alone.  Plus (``shared`` [T, W], a tensor or split sums, given)
     sigmoid(logits[t, shared_gate_col]) * shared[t] (``shared_gate_col`` negative: plus shared[t]).  ``w_gate_up`` [E, 2F, W] (an expert's gate rows,
     then its up rows), ``w_down`` [E, W, F], both of x's type.  The (token, expert) pairs are sorted by
     expert on the device into tiles of EXPERT_TILE_ROWS (or EXPERT_TILE_ROWS_LARGE) rows of one expert; a
@@ -1445,8 +1622,10 @@ def routed_experts(x: torch.Tensor, ids, weights, w_gate_up: torch.Tensor,
     _need(w_down, "w_down", x.dtype, 3)
     t, w = x.shape
     n_exp, two_f, w2 = w_gate_up.shape
-    f = two_f // 2
-    if w2 != w or tuple(w_down.shape) != (n_exp, w, f) or two_f != 2 * f or ids.shape[0] != t \
+    f = two_f // 2 if gated else two_f
+    if limited is not None and not gated:
+        raise KernelError("routed_experts: experts without a gate have no limited gate")
+    if w2 != w or tuple(w_down.shape) != (n_exp, w, f) or (gated and two_f != 2 * f) or ids.shape[0] != t \
             or (weights is not None and tuple(weights.shape) != (t, top)):
         raise KernelError(f"routed_experts: x {tuple(x.shape)}, gate/up {tuple(w_gate_up.shape)}, down "
                           f"{tuple(w_down.shape)}, ids {tuple(ids.shape)}")
@@ -1454,7 +1633,7 @@ def routed_experts(x: torch.Tensor, ids, weights, w_gate_up: torch.Tensor,
     dev = x.device
     pairs = t * top
     on_tc = EXPERTS_TC and x.dtype == torch.bfloat16 and pairs >= EXPERT_TILE_ROWS_TC * n_exp \
-        and f % 128 == 0 and w % 256 == 0 and x.is_contiguous()
+        and f % (128 if gated else 256) == 0 and w % 256 == 0 and x.is_contiguous()
     tile = EXPERT_TILE_ROWS_TC if on_tc \
         else EXPERT_TILE_ROWS_LARGE if pairs >= EXPERT_TILE_ROWS_LARGE * n_exp else EXPERT_TILE_ROWS
     max_tiles = pairs // tile + min(n_exp, pairs) + 1
@@ -1473,7 +1652,7 @@ def routed_experts(x: torch.Tensor, ids, weights, w_gate_up: torch.Tensor,
         _check(st, "routed_experts(rows in the experts' order)")
         hidden = torch.empty(rows, f, dtype=x.dtype, device=dev)
         st = large.dib_gemm_bf16_large_grouped(_ptr(sorted_x), _ptr(w_gate_up), _ptr(hidden), c_int(rows), c_int(f),
-                                               c_int(w), c_int(1), c_int(0), tile_expert, c_int(n_exp),
+                                               c_int(w), c_int(1 if gated else 2), c_int(0), tile_expert, c_int(n_exp),
                                                c_float(limit), c_float(alpha), c_int(_sms(dev)), _stream())
         _check(st, "routed_experts(gate and up, tcgen05)", f"rows {rows}, F {f}, W {w}")
         sorted_y = torch.empty(rows, w, dtype=torch.float32, device=dev)
@@ -1485,9 +1664,13 @@ def routed_experts(x: torch.Tensor, ids, weights, w_gate_up: torch.Tensor,
         _check(st, "routed_experts(rows back to their pairs)")
     else:
         hidden = torch.empty(max_tiles * tile, f, dtype=x.dtype, device=dev)
-        st = lib.dib_moe_gate_up(_ptr(x), c_int(_dt(x, "x")), _ptr(order), c_int(max_tiles), c_int(tile), c_int(top),
-                                 _ptr(w_gate_up), _ptr(hidden), c_int(f), c_int(w), c_float(limit), c_float(alpha),
-                                 _stream())
+        if gated:
+            st = lib.dib_moe_gate_up(_ptr(x), c_int(_dt(x, "x")), _ptr(order), c_int(max_tiles), c_int(tile), c_int(top),
+                                     _ptr(w_gate_up), _ptr(hidden), c_int(f), c_int(w), c_float(limit), c_float(alpha),
+                                     _stream())
+        else:
+            st = lib.dib_moe_up(_ptr(x), c_int(_dt(x, "x")), _ptr(order), c_int(max_tiles), c_int(tile), c_int(top),
+                                _ptr(w_gate_up), _ptr(hidden), c_int(f), c_int(w), _stream())
         _check(st, "routed_experts(gate and up)")
         st = lib.dib_moe_down(_ptr(hidden), c_int(_dt(x, "x")), _ptr(order), c_int(max_tiles), c_int(tile), _ptr(w_down),
                               _ptr(per_pair), c_int(f), c_int(w), _stream())
@@ -1549,13 +1732,14 @@ def _cache_pages(kv_cache, page_elems: int, what: str) -> int:
 def attn_prepare(proj, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int, q_norm_weight,
                  k_norm_weight, eps: float, freq, rotary_dim: int, positions: torch.Tensor, kv_cache,
                  slot_mapping, page_size: int, out_dtype, bias=None, norm_scope: str = "head",
-                 rotary_layout: str = "halves", conv_weight=None, conv_state=None, step=None) -> torch.Tensor:
+                 rotary_layout: str = "halves", conv_weight=None, conv_state=None, step=None,
+                 amplitude: float = 1.0) -> torch.Tensor:
     """From each token's projection row [q heads | k heads | v heads | anything else] (plus ``bias``,
     float32 over q, k and v, when given): RMS norm of q and k (when a weight is given; ``norm_scope``
     "head": per head, weights of head_dim elements; "projection": over all of q's (k's) heads at once,
     weights of that many elements), rotation of the first ``rotary_dim`` elements of each head by the
     token's position (``rotary_layout`` "halves": element i with i + rotary_dim / 2, "pairs": element 2i
-    with 2i + 1; angle = position * freq[i], float32), q [T, Hq, D] returned, k and v to the token's slot
+    with 2i + 1; angle = position * freq[i], float32, cosine and sine times ``amplitude``), q [T, Hq, D] returned, k and v to the token's slot
     of the paged cache (a page: keys [Hkv, page_size, D], then values [Hkv, page_size, Dv]).
     ``conv_weight`` (float32 [q + k + v channels, taps], the last tap the current token's): each channel
     of q, k and v first passes a causal convolution over its sequence's tokens, before norm and rotation;
@@ -1612,7 +1796,7 @@ def attn_prepare(proj, num_heads: int, num_kv_heads: int, head_dim: int, v_head_
             _ptr(k_norm_weight), c_int(1 if whole else 0), c_float(eps), _ptr(freq),
             c_int(rotary_dim if freq is not None else 0), c_int(1 if rotary_layout == "pairs" else 0), _ptr(positions),
             _ptr(slot_mapping), c_int(t), c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(v_head_dim),
-            c_int(page_size), c_longlong(num_pages), c_int(_DT[out_dtype]), *conv_args, _stream())
+            c_int(page_size), c_longlong(num_pages), c_int(_DT[out_dtype]), *conv_args, c_float(amplitude), _stream())
         _check(st, "attn_prepare(row)", f"heads {num_heads}/{num_kv_heads} of {head_dim}/{v_head_dim}",
                kernels=2 if conv_weight is not None and conv_weight.shape[1] > 1 else 1)
         return q
@@ -1620,7 +1804,7 @@ def attn_prepare(proj, num_heads: int, num_kv_heads: int, head_dim: int, v_head_
         *_source_args(proj), c_longlong(width), _ptr(q), _ptr(kv_cache), _ptr(q_norm_weight), _ptr(k_norm_weight),
         c_float(eps), _ptr(freq), c_int(rotary_dim if freq is not None else 0), _ptr(positions),
         _ptr(slot_mapping), c_int(t), c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(v_head_dim),
-        c_int(page_size), c_longlong(num_pages), c_int(_DT[out_dtype]), _stream())
+        c_int(page_size), c_longlong(num_pages), c_int(_DT[out_dtype]), c_float(amplitude), _stream())
     _check(st, "attn_prepare", f"heads {num_heads}/{num_kv_heads} of {head_dim}/{v_head_dim}")
     return q
 
@@ -1662,6 +1846,55 @@ def latent_prepare(proj, num_heads: int, plain_dim: int, rot_dim: int, rank: int
         c_int(1 if rotary_layout == "pairs" else 0), c_float(amplitude), _stream())
     _check(st, "latent_prepare")
     return q
+
+
+def latent_rows(proj, q_col: int, q_rank: int, q_norm_weight: torch.Tensor, kv_col: int, rank: int, rot_dim: int,
+                latent_norm_weight: torch.Tensor, eps: float, freq, positions, kv_cache, slot_mapping, page_size: int,
+                out_dtype, rotary_layout: str = "halves", amplitude: float = 1.0) -> torch.Tensor:
+    """From each token's projection row: the query latent (``q_rank`` elements at column ``q_col``), RMS-normed
+    with its weight, is returned [T, q_rank]; the key/value latent (``rank`` elements at column ``kv_col``),
+    RMS-normed with its weight, goes to the token's cache row [rank + rot_dim], behind it the rotated key part
+    (the ``rot_dim`` elements after the latent; 0: there is none).  ``kv_cache`` None: nothing is stored."""
+    t, width = proj.shape
+    for w, name, n in ((q_norm_weight, "q_norm_weight", q_rank), (latent_norm_weight, "latent_norm_weight", rank)):
+        _need(w, name, torch.float32, 1)
+        if w.shape[0] != n:
+            raise KernelError(f"latent_rows: {name} has {w.shape[0]} elements for a latent of {n}")
+    if q_col + q_rank > width or kv_col + rank + rot_dim > width or rotary_layout not in ("halves", "pairs"):
+        raise KernelError(f"latent_rows: rows of {width} elements, rotary layout {rotary_layout!r}")
+    if rot_dim:
+        _need(freq, "freq", torch.float32, 1)
+        if freq.shape[0] * 2 != rot_dim:
+            raise KernelError(f"latent_rows: {freq.shape[0]} frequencies for {rot_dim} rotated elements")
+    _need(positions, "positions", torch.int32, 1)
+    num_pages = 0
+    if kv_cache is not None:
+        _need(kv_cache, "kv_cache", out_dtype)
+        _need(slot_mapping, "slot_mapping", torch.int32, 1)
+        num_pages = _cache_pages(kv_cache, page_size * (rank + rot_dim), "latent_rows")
+    q = torch.empty(t, q_rank, dtype=out_dtype, device=proj.device)
+    st = _lib("masked_attention").dib_latent_rows(
+        *_source_args(proj), c_longlong(width), c_longlong(q_col), c_int(q_rank), _ptr(q_norm_weight), _ptr(q),
+        c_longlong(kv_col), c_int(rank), c_int(rot_dim), _ptr(latent_norm_weight), _ptr(kv_cache), c_float(eps),
+        _ptr(freq if rot_dim else None), _ptr(positions), _ptr(slot_mapping), c_int(t), c_int(page_size),
+        c_longlong(num_pages), c_int(_DT[out_dtype]), c_int(1 if rotary_layout == "pairs" else 0), c_float(amplitude),
+        _stream())
+    _check(st, "latent_rows")
+    return q
+
+
+def sigmoid_gate_(x: torch.Tensor, gate, gate_col: int, per: int = 1) -> torch.Tensor:
+    """In place: x[t, c] *= sigmoid(gate[t, gate_col + c / per]), float32 arithmetic; ``gate`` a tensor or split
+    sums, ``per`` neighbouring elements share a gate number."""
+    _need(x, "x", None, 2)
+    t, width = x.shape
+    if gate.shape[0] != t or per < 1 or width % per or gate.shape[1] < gate_col + width // per:
+        raise KernelError(f"sigmoid_gate_: gate of shape {tuple(gate.shape)} from column {gate_col} for {(t, width)}")
+    st = _lib("masked_attention").dib_sigmoid_gate_(
+        _ptr(x), *_source_args(gate), c_longlong(gate.shape[1]), c_longlong(gate_col), c_int(t), c_int(width),
+        c_int(per), c_int(_dt(x, "x")), _stream())
+    _check(st, "sigmoid_gate_")
+    return x
 
 
 def heads_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -1709,12 +1942,13 @@ HEADS_LINEAR_LIBRARY_ROWS = int(__import__("os").environ.get("DIB200_HEADS_LINEA
 def masked_attention(q: torch.Tensor, kv_cache: torch.Tensor, meta, scale: float, num_kv_heads: int,
                      v_head_dim: int, page_size: int, mask: str = "causal", mask_size=None, sink=None,
                      gate=None, gate_col: int = 0, values_in_keys: bool = False, keep_first: int = 0,
-                     softcap=None) -> torch.Tensor:
+                     softcap=None, gate_per_head: bool = False) -> torch.Tensor:
     """[T, Hq, Dv]: softmax attention of every token of the step over the keys of its sequence in the
     paged cache that ``mask`` lets it see (a query at position p: "causal" 0 .. p; "window" p - size + 1
     .. p, and with ``keep_first`` also the keys 0 .. keep_first - 1; "chunk" floor(p / size) * size .. p).  ``sink`` float32 [Hq]: the denominator also holds
     exp(sink[h]) as one more term that brings nothing into the output and is taken as it is.  ``gate`` [T, >= gate_col + Hq * Dv] (a tensor or split
-    sums): the output is multiplied by sigmoid(gate[t, gate_col + h * Dv + d]).  ``values_in_keys``: the
+    sums): the output is multiplied by sigmoid(gate[t, gate_col + h * Dv + d]) (``gate_per_head``: sigmoid(gate[t,
+    gate_col + h])).  ``values_in_keys``: the
     cache holds keys only and a key's first Dv elements are its value.  ``softcap`` c: a score (after the
     scale) becomes c * tanh(score / c) before the softmax."""
     cap = 0.0 if softcap is None else float(softcap)
@@ -1737,7 +1971,7 @@ def masked_attention(q: torch.Tensor, kv_cache: torch.Tensor, meta, scale: float
             raise KernelError(f"masked_attention: {sink.shape[0]} sinks for {hq} heads")
     gate_args, gate_row = (c_void_p(0), c_int(0), c_int(1), c_longlong(0)), 0
     if gate is not None:
-        if gate.shape[0] != t or gate.shape[1] < gate_col + hq * v_head_dim:
+        if gate.shape[0] != t or gate.shape[1] < gate_col + (hq if gate_per_head else hq * v_head_dim):
             raise KernelError(f"masked_attention: gate of shape {tuple(gate.shape)}")
         gate_args, gate_row = _source_args(gate), gate.shape[1]
     _need(meta.block_table, "block_table", torch.int32, 2)
@@ -1756,10 +1990,7 @@ def masked_attention(q: torch.Tensor, kv_cache: torch.Tensor, meta, scale: float
             cache5 = kv_cache.view(kv_cache.shape[0], 2, num_kv_heads, page_size, dk)
             attention_bf16.run(q, out, cache5, meta, scale, {0: 0, 1: size, 2: -size}[kind], False, sink)
             if gate is not None:
-                st = _lib("masked_attention").dib_sigmoid_gate_(
-                    _ptr(out), *gate_args, c_longlong(gate_row), c_longlong(gate_col), c_int(t),
-                    c_int(hq * v_head_dim), c_int(_dt(q, "q")), _stream())
-                _check(st, "sigmoid_gate_")
+                sigmoid_gate_(out.view(t, hq * v_head_dim), gate, gate_col, v_head_dim if gate_per_head else 1)
             return out
     group = hq // num_kv_heads
     if q.dtype == torch.bfloat16 and MASKED_ATTENTION_TC and MASKED_ATTENTION_MMA and dk % 16 == 0 and v_head_dim % 16 == 0 \
@@ -1801,7 +2032,7 @@ def masked_attention(q: torch.Tensor, kv_cache: torch.Tensor, meta, scale: float
                     c_int(tiles.shape[0]), _ptr(sink),
                     c_int(hq), c_int(num_kv_heads), c_int(dk), c_int(v_head_dim), c_int(dv_stored),
                     c_int(page_size), c_float(scale), c_int(kind), c_int(size), c_int(keep), *gate_args,
-                    c_longlong(gate_row), c_longlong(gate_col), c_int(form_rows), _ptr(part_o), _ptr(part_ml),
+                    c_longlong(gate_row), c_longlong(gate_col), c_int(1 if gate_per_head else 0), c_int(form_rows), _ptr(part_o), _ptr(part_ml),
                     c_int(MASKED_DECODE_CHUNK_TILES), c_int(max_chunks), c_int(n_dec), c_float(cap), _stream())
                 _check(st, "masked_attention(tensor cores)", f"heads {hq}/{num_kv_heads}, sizes {dk}/{v_head_dim}",
                        kernels=2 if part_o is not None else 1)
@@ -1810,7 +2041,8 @@ def masked_attention(q: torch.Tensor, kv_cache: torch.Tensor, meta, scale: float
         _ptr(q), _ptr(out), _ptr(kv_cache), _ptr(meta.block_table), c_int(meta.block_table.shape[1]),
         _ptr(meta.token_seq), _ptr(meta.positions), c_int(t), c_int(hq), c_int(num_kv_heads), c_int(dk),
         c_int(v_head_dim), c_int(dv_stored), c_int(page_size), c_float(scale), c_int(kind), c_int(size), c_int(keep),
-        _ptr(sink), *gate_args, c_longlong(gate_row), c_longlong(gate_col), c_int(_dt(q, "q")), c_float(cap),
+        _ptr(sink), *gate_args, c_longlong(gate_row), c_longlong(gate_col), c_int(1 if gate_per_head else 0),
+        c_int(_dt(q, "q")), c_float(cap),
         _stream())
     _check(st, "masked_attention", f"heads {hq}/{num_kv_heads}, sizes {dk}/{v_head_dim}")
     return out

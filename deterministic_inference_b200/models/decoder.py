@@ -12,8 +12,8 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from ..parts import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, STREAM_ADDENDS, BuildContext,
-                     ModelPlan, TensorSpec)
+from ..parts import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, STREAM_ADDENDS, STREAM_ENTRIES,
+                     BuildContext, ModelPlan, TensorSpec)
 
 
 class DecoderModel:
@@ -39,6 +39,9 @@ class DecoderModel:
         self.head = HEADS.build(plan.head, self.ctx)
         self.stream_addend = None if plan.stream_addend is None \
             else STREAM_ADDENDS.build(plan.stream_addend, self.ctx)
+        self.stream_entry = None if plan.stream_entry is None \
+            else STREAM_ENTRIES.build(plan.stream_entry, self.ctx)
+        self.last_entry = max((i for i, e in enumerate(plan.schedule) if e.enters), default=-1)
 
     # ---- weights ------------------------------------------------------------
 
@@ -52,6 +55,8 @@ class DecoderModel:
             yield from getattr(b, "extra_parts", ())
         if self.stream_addend is not None:
             yield self.stream_addend
+        if self.stream_entry is not None:
+            yield self.stream_entry
         yield self.final_norm
         yield self.head
 
@@ -118,7 +123,10 @@ class DecoderModel:
         else:
             hidden = self.embedding.forward(step.input_ids)
         residual = None
-        for e in self.plan.schedule:
+        kept = self.stream_entry.start(hidden) if self.last_entry >= 0 else None
+        for i, e in enumerate(self.plan.schedule):
+            if e.enters:
+                hidden, residual = self.stream_entry.enter(hidden, residual, kept, last=i == self.last_entry)
             if e.enter_vector is not None:
                 # (float32 additions: whether the vector or the pending output joins the stream first
                 # is a matter of rounding alone)

@@ -17,6 +17,7 @@ import torch
 
 from ..config.bovitar_config import BovitarConfig
 from ..config.gamilorn_config import GamilornConfig
+from ..config.gikarax_config import GikaraxConfig
 from ..config.kipezen_config import KipezenConfig
 from ..config.model_config import Qwen3Config
 from ..config.nedupel_config import NedupelConfig
@@ -41,6 +42,7 @@ register_architecture("Zatirax", ZatiraxConfig)
 register_architecture("Kipezen", KipezenConfig)
 register_architecture("Bovitar", BovitarConfig)
 register_architecture("Nedupel", NedupelConfig)
+register_architecture("Gikarax", GikaraxConfig)
 
 
 def config_from_dir(model_dir):

@@ -66,6 +66,30 @@ class PreNormStreamBlock(Block):
         return hidden, residual
 
 
+@register_block("parallel_f32_stream")
+class ParallelStreamBlock(Block):
+    """ONE norm whose output both sublayers read, the residual stream in float32: with h = norm(x),
+    x <- x + (mixer(h) + feed_forward(h)).  Both outputs are handed on as one pending sum, which the stream's
+    next reader adds up in float32; ``feed_forward_norm`` is not used (kind "none").  A layer without a
+    feed-forward (kind "none") hands on its mixer's output."""
+
+    def __init__(self, ctx, mixer, feed_forward, mixer_norm, feed_forward_norm):
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
+
+    def forward(self, hidden, residual, step, cache):
+        if residual is None:
+            residual = hidden
+            h = self.mixer_norm.forward(residual)
+        else:
+            h, residual = self.mixer_norm.add_forward(hidden, residual)
+        mixed = self.mixer.forward(h, step, cache)
+        if self.feed_forward.kind == "none":
+            return mixed, residual
+        terms = mixed.terms if isinstance(mixed, ops.WeightedSum) else [(1.0, mixed)]
+        return ops.WeightedSum([*terms, (1.0, self.feed_forward.run(h, step))]), residual
+
+
 @register_block("sandwich_f32_stream")
 class SandwichStreamBlock(Block):
     """A norm in front of and behind each sublayer, the residual stream in float32:

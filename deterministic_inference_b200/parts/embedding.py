@@ -11,7 +11,7 @@ import torch
 
 from ..kernels import ops
 from .base import Head, Part, TokenEmbedding
-from .registry import register_embedding, register_head, register_stream_addend
+from .registry import register_embedding, register_head, register_stream_addend, register_stream_entry
 from .spec import TensorSpec
 
 
@@ -105,6 +105,39 @@ class RowVectors(Part):
         if not 0 <= index < self.count:
             raise IndexError(f"{self.name}: vector {index} of {self.count}")
         return ops.stream_add_(stream, bias=self.vectors[index])
+
+
+@register_stream_entry("mix_with_start")
+class MixWithStart(Part):
+    """The stream x becomes W [x; x0], x0 the stream as the embedding left it, W [width, 2 width] with x's
+    columns first.  W's two halves are separate products: ``start`` runs x0's once a step, and ``enter``
+    returns x's product as the pending term of a stream that starts as x0's, so nothing is rounded between
+    them and each further entry costs half a product."""
+
+    def __init__(self, ctx, name: str, hidden_size: int):
+        self.name, self.hidden_size = name, int(hidden_size)
+        self.dtype = ctx.dtype
+        self.w_stream = self.w_start = None
+
+    def tensor_specs(self):
+        return [TensorSpec(self.name, (self.hidden_size, 2 * self.hidden_size))]
+
+    def load(self, tensors):
+        w = tensors[self.name]
+        self.w_stream = w[:, :self.hidden_size].contiguous()
+        self.w_start = w[:, self.hidden_size:].contiguous()
+
+    def start(self, stream):
+        """What ``enter`` keeps of the embedding's output (float32 [T, width])."""
+        return ops.as_tensor(ops.linear(ops.stream_read(stream, None, self.dtype), self.w_start,
+                                        out_dtype=torch.float32))
+
+    def enter(self, hidden, residual, kept, last: bool):
+        """(pending term, stream) after the entry; ``last``: no later entry of the step needs ``kept``."""
+        if residual is None:
+            residual, hidden = hidden, None
+        y = ops.linear(ops.stream_read(residual, hidden, self.dtype), self.w_stream, out_dtype=torch.float32)
+        return y, kept if last else kept.clone()
 
 
 @register_head("linear_head")

@@ -18,6 +18,11 @@ shows ("causal", "window", "chunk" as in ``masked_attention``); norms, angles, s
 are float32.  ``rotary_layout``: "halves" (element i of a rotated part turns with i + rot_dim / 2) or
 "pairs" (2i with 2i + 1); the position encoding's ``amplitude`` multiplies cosine and sine.
 
+``rot_dim`` 0 (no position encoding): there is no rotated part, the cache row is the latent alone.
+``q_rank``: the queries go through a latent of their own, q = W_uq c_q with c_q = RMS norm of W_dq x with a
+weight.  ``gate``: the heads' values side by side are multiplied element by element with sigmoid(W_g x)
+before the output projection.
+
 ``own_latent`` off: the layer has no W_dkv and reads the rows that another layer of the same
 kv_rank, rot_dim and rotation left in the cache its schedule entry names.
 """
@@ -37,9 +42,10 @@ from .spec import PagedKVSpec, PartSpec, TensorSpec
 @register_mixer("latent_attention")
 class LatentAttention(Mixer):
     def __init__(self, ctx, prefix: str, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int,
-                 v_head_dim: int, kv_rank: int, scale: float, position_encoding: PartSpec, norm_eps: float,
+                 v_head_dim: int, kv_rank: int, scale: float, position_encoding: Optional[PartSpec], norm_eps: float,
                  mask: str = "causal", mask_size: Optional[int] = None, names: Optional[dict] = None,
-                 rotary_layout: str = "halves", own_latent: bool = True):
+                 rotary_layout: str = "halves", own_latent: bool = True, q_rank: Optional[int] = None,
+                 gate: bool = False):
         if mask not in ("causal", "window", "chunk"):
             raise ValueError(f"mask {mask!r} is not known ('causal', 'window', 'chunk')")
         if mask != "causal" and (mask_size is None or int(mask_size) < 1):
@@ -52,19 +58,33 @@ class LatentAttention(Mixer):
         self.head_dim, self.rot_dim, self.v_head_dim = int(head_dim), int(rot_dim), int(v_head_dim)
         self.kv_rank, self.scale, self.norm_eps = int(kv_rank), float(scale), float(norm_eps)
         self.mask, self.mask_size = mask, None if mask == "causal" else int(mask_size)
-        self.names = dict(q="q", down="dkv", latent_norm="dkv.norm", key_map="uk", value_map="uv", o="o")
+        self.q_rank, self.gate = None if q_rank is None else int(q_rank), bool(gate)
+        if not self.own_latent and (self.q_rank is not None or self.rot_dim == 0):
+            raise ValueError("latent_attention: a layer that reads another's rows has plain queries and a rotated part")
+        self.names = dict(q="q", down="dkv", latent_norm="dkv.norm", key_map="uk", value_map="uv", o="o", q_down="dq",
+                          q_norm="dq.norm", q_up="uq", gate="g")
         self.names.update(names or {})
-        self.position_encoding = POSITION_ENCODINGS.build(position_encoding, ctx)
-        if self.position_encoding.rotary_dim != self.rot_dim:
-            raise ValueError(f"latent_attention: the rotation covers {self.position_encoding.rotary_dim} "
+        self.position_encoding = None if position_encoding is None or not self.rot_dim \
+            else POSITION_ENCODINGS.build(position_encoding, ctx)
+        if getattr(self.position_encoding, "rotary_dim", 0) != self.rot_dim:
+            raise ValueError(f"latent_attention: the rotation covers {getattr(self.position_encoding, 'rotary_dim', 0)} "
                              f"elements, the rotated part has {self.rot_dim}")
+        self.amplitude = getattr(self.position_encoding, "amplitude", 1.0)
         self.out_dtype = ctx.dtype
         self.w_in = self.w_key = self.w_value = self.w_o = self.latent_norm = self.freq = None
+        self.w_q_up = self.q_norm = None
 
     def tensor_specs(self):
         p, n, w = self.prefix, self.names, self.hidden_size
         h, d, r, e, c = self.num_heads, self.head_dim, self.rot_dim, self.v_head_dim, self.kv_rank
-        specs = [TensorSpec(p + n["q"], (h * (d + r), w))]
+        if self.q_rank is None:
+            specs = [TensorSpec(p + n["q"], (h * (d + r), w))]
+        else:
+            specs = [TensorSpec(p + n["q_down"], (self.q_rank, w)),
+                     TensorSpec(p + n["q_norm"], (self.q_rank,), role="vector", init="one_plus_normal"),
+                     TensorSpec(p + n["q_up"], (h * (d + r), self.q_rank))]
+        if self.gate:
+            specs.append(TensorSpec(p + n["gate"], (h * e, w)))
         if self.own_latent:
             specs += [TensorSpec(p + n["down"], (c + r, w)),
                       TensorSpec(p + n["latent_norm"], (c,), role="vector", init="one_plus_normal")]
@@ -74,17 +94,23 @@ class LatentAttention(Mixer):
     def load(self, tensors):
         p, n = self.prefix, self.names
         h, d, e, c = self.num_heads, self.head_dim, self.v_head_dim, self.kv_rank
+        # one product gives [queries, or their latent | latent, rotated key part | gate]
+        rows = [tensors[p + n["q" if self.q_rank is None else "q_down"]]]
         if self.own_latent:
-            self.w_in = torch.cat([tensors[p + n["q"]], tensors[p + n["down"]]], dim=0).contiguous()
+            rows.append(tensors[p + n["down"]])
             self.latent_norm = tensors[p + n["latent_norm"]]
-        else:
-            self.w_in = tensors[p + n["q"]]
+        if self.gate:
+            rows.append(tensors[p + n["gate"]])
+        self.w_in = torch.cat(rows, dim=0).contiguous() if len(rows) > 1 else rows[0]
+        if self.q_rank is not None:
+            self.q_norm, self.w_q_up = tensors[p + n["q_norm"]], tensors[p + n["q_up"]]
         # per head [K, N]: the key map takes a query's plain part [d] to the latent's size [c]; the
         # value map takes a weighted latent [c] to the head's value [e]
         self.w_key = tensors[p + n["key_map"]].view(h, d, c).contiguous()
         self.w_value = tensors[p + n["value_map"]].view(h, e, c).transpose(1, 2).contiguous()
         self.w_o = tensors[p + n["o"]]
-        self.freq = self.position_encoding.frequencies()
+        if self.rot_dim:
+            self.freq = self.position_encoding.frequencies()
 
     def cache_spec(self):
         return PagedKVSpec(1, self.kv_rank + self.rot_dim, self.mask_size, v_head_dim=0,
@@ -92,15 +118,32 @@ class LatentAttention(Mixer):
 
     def forward(self, x, step, cache):
         h, d, r, e, c = self.num_heads, self.head_dim, self.rot_dim, self.v_head_dim, self.kv_rank
-        proj = ops.as_tensor(ops.linear(x, self.w_in))
+        proj = ops.linear(x, self.w_in)
         t, width = proj.shape
-        q = ops.latent_prepare(proj, h, d, r, c, self.latent_norm, self.norm_eps, self.freq, step.positions,
-                               cache.kv if cache.writes and self.own_latent else None, cache.slot_mapping,
-                               cache.page_size, self.out_dtype, rotary_layout=self.rotary_layout,
-                               amplitude=self.position_encoding.amplitude)
-        ops.heads_linear(proj.as_strided((t, h, d), (width, d + r, 1)), self.w_key, q[:, :, :c])
+        stored = cache.kv if cache.writes and self.own_latent else None
+        rotation = dict(rotary_layout=self.rotary_layout, amplitude=self.amplitude)
+        nq = h * (d + r)
+        gate_col = (nq if self.q_rank is None else self.q_rank) + (c + r if self.own_latent else 0)
+        if self.q_rank is not None:
+            # the two latents, then the queries out of theirs
+            c_q = ops.latent_rows(proj, 0, self.q_rank, self.q_norm, self.q_rank, c, r, self.latent_norm, self.norm_eps,
+                                  self.freq, step.positions, stored, cache.slot_mapping, cache.page_size, self.out_dtype,
+                                  **rotation)
+            heads = ops.as_tensor(ops.linear(c_q, self.w_q_up))
+            q = torch.empty(t, h, c, dtype=heads.dtype, device=heads.device) if r == 0 else \
+                ops.latent_prepare(heads, h, d, r, c, None, self.norm_eps, self.freq, step.positions, None,
+                                   cache.slot_mapping, cache.page_size, self.out_dtype, **rotation)
+        else:
+            heads = proj = ops.as_tensor(proj)
+            q = ops.latent_prepare(proj, h, d, r, c, self.latent_norm, self.norm_eps, self.freq, step.positions, stored,
+                                   cache.slot_mapping, cache.page_size, self.out_dtype, **rotation)
+        row = heads.shape[1]
+        ops.heads_linear(heads.as_strided((t, h, d), (row, d + r, 1)), self.w_key, q[:, :, :c])
         latent = ops.masked_attention(q, cache.kv, cache.attention_meta, self.scale, 1, c, cache.page_size,
                                       self.mask, self.mask_size, values_in_keys=True)
-        o = torch.empty(t, h, e, dtype=proj.dtype, device=proj.device)
+        o = torch.empty(t, h, e, dtype=heads.dtype, device=heads.device)
         ops.heads_linear(latent, self.w_value, o)
-        return ops.linear(o.view(t, h * e), self.w_o)
+        o = o.view(t, h * e)
+        if self.gate:
+            ops.sigmoid_gate_(o, proj, gate_col)
+        return ops.linear(o, self.w_o)

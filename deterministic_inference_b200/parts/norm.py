@@ -61,6 +61,30 @@ class StreamRMSNorm(Norm):
         return ops.stream_rms_norm(residual, self.weight, self.eps, self.out_dtype, add=x), residual
 
 
+@register_norm("stream_layer_norm")
+class StreamLayerNorm(Norm):
+    """Layer norm of a residual stream that is kept in float32 whatever the engine's storage type:
+    y = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * w, no bias, written in the engine's type.
+    ``add_forward`` first adds whatever term is pending to the stream, in float32 and in place."""
+
+    def __init__(self, ctx, name: str, size: int, eps: float):
+        self.name, self.size, self.eps = name, int(size), float(eps)
+        self.out_dtype = ctx.dtype
+        self.weight = None
+
+    def tensor_specs(self):
+        return [TensorSpec(self.name, (self.size,), role="vector", init="one_plus_normal")]
+
+    def load(self, tensors):
+        self.weight = tensors[self.name]
+
+    def forward(self, x):
+        return ops.stream_layer_norm(x, self.weight, self.eps, self.out_dtype)
+
+    def add_forward(self, x, residual):
+        return ops.stream_layer_norm(residual, self.weight, self.eps, self.out_dtype, add=x), residual
+
+
 @register_norm("stream_post_norm")
 class StreamPostNorm(Norm):
     """RMSNorm of a part's OUTPUT on its way into a float32 residual stream:

@@ -62,6 +62,7 @@ NORMS = Registry("norm")
 POSITION_ENCODINGS = Registry("position encoding")
 BLOCKS = Registry("block")
 STREAM_ADDENDS = Registry("stream addend")     # what a schedule entry may add to the stream on entry
+STREAM_ENTRIES = Registry("stream entry")      # what a schedule entry may replace the stream by on entry
 
 register_embedding = EMBEDDINGS.register
 register_head = HEADS.register
@@ -71,3 +72,4 @@ register_norm = NORMS.register
 register_position_encoding = POSITION_ENCODINGS.register
 register_block = BLOCKS.register
 register_stream_addend = STREAM_ADDENDS.register
+register_stream_entry = STREAM_ENTRIES.register

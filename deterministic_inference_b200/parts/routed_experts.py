@@ -2,11 +2,14 @@
 
 ``num_experts`` gated feed-forwards (W_down act(W_gate x, W_up x), no biases), of which each
 token uses ``top``.  ``activation`` "silu": silu(g) u; "limited_swish": with g = min(g, limit) and u =
-clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1).  ``score`` "table": no router; row i of a stored
+clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1); "gelu": experts without a gate matrix, W_down gelu(W_up x)
+with the erf gelu.  ``score`` "table": no router; row i of a stored
 integer table [vocabulary, top] names the experts of token id i, all weighted ``route_scale`` / top.
 Otherwise, router: z = W_router x in float32, scores s = sigmoid(z) or (``score``
 "softmax") softmax(z) over all experts.  The choice is made on s + correction (a stored vector),
-the weights use s without it.  The experts form ``group_count`` equal groups of neighbours; a
+the weights use s without it; ``correction`` off: there is none.  ``score`` "chosen_softmax": the choice is made
+on z (+ correction), and s of a chosen expert is exp(z), so that the weights are the softmax over the chosen
+logits alone.  The experts form ``group_count`` equal groups of neighbours; a
 group's score is the sum of its ``group_top`` largest choice scores (2, or 1: its largest), and only
 experts of the ``group_keep`` best groups can be chosen (the others count as minus infinity).  The
 ``top`` largest choice scores win; their weights are their scores s over the sum of those
@@ -34,12 +37,16 @@ class RoutedExperts(FeedForward):
                  shared_intermediate_size: Optional[int] = None, weight_eps: float = 1e-20,
                  names: Optional[dict] = None, score: str = "sigmoid", group_top: int = 2, normalize: bool = True,
                  shared_gate: bool = True, activation: str = "silu", limit: Optional[float] = None,
-                 alpha: float = 1.702, vocab_size: Optional[int] = None):
+                 alpha: float = 1.702, vocab_size: Optional[int] = None, correction: bool = True):
         if (score != "table" and score not in ops.ROUTER_SCORES) or int(group_top) not in (1, 2):
             raise ValueError(f"routed_experts: score {score!r} ({sorted(ops.ROUTER_SCORES)}, 'table') or group_top "
                              f"{group_top!r} (1, 2) is not known")
-        if activation not in ("silu", "limited_swish"):
-            raise ValueError(f"routed_experts: activation {activation!r} has no kernel ('silu', 'limited_swish')")
+        if activation not in ("silu", "limited_swish", "gelu"):
+            raise ValueError(f"routed_experts: activation {activation!r} has no kernel ('silu', 'limited_swish', 'gelu')")
+        if activation == "gelu" and shared_intermediate_size is not None:
+            raise ValueError("routed_experts: a shared expert has a gate ('silu', 'limited_swish')")
+        if score == "chosen_softmax" and not normalize:
+            raise ValueError("routed_experts: the softmax over the chosen logits is a normalized score")
         if activation == "limited_swish" and (limit is None or not float(limit) > 0):
             raise ValueError("routed_experts: 'limited_swish' needs a positive limit")
         if score == "table" and (vocab_size is None or shared_gate and shared_intermediate_size is not None
@@ -57,6 +64,7 @@ class RoutedExperts(FeedForward):
         self.shared_size = None if shared_intermediate_size is None else int(shared_intermediate_size)
         self.score, self.group_top, self.normalize = score, int(group_top), bool(normalize)
         self.shared_gate = bool(shared_gate) and self.shared_size is not None
+        self.gated, self.has_correction = activation != "gelu", bool(correction)
         self.limited = (float(limit), float(alpha)) if activation == "limited_swish" else None
         self.vocab_size = None if vocab_size is None else int(vocab_size)
         self.needs_step = score == "table"          # the choice is made on the step's token ids
@@ -72,14 +80,16 @@ class RoutedExperts(FeedForward):
         specs = []
         for e in range(self.num_experts):
             q = p + n["expert"].format(e)
-            specs += [TensorSpec(q + n["gate"], (f, w)), TensorSpec(q + n["up"], (f, w)),
-                      TensorSpec(q + n["down"], (w, f))]
+            if self.gated:
+                specs.append(TensorSpec(q + n["gate"], (f, w)))
+            specs += [TensorSpec(q + n["up"], (f, w)), TensorSpec(q + n["down"], (w, f))]
         if self.score == "table":
             specs.append(TensorSpec(p + n["table"], (self.vocab_size, self.top), role="index", init="distinct",
                                     high=self.num_experts))
         else:
-            specs += [TensorSpec(p + n["router"], (self.num_experts, w)),
-                      TensorSpec(p + n["correction"], (self.num_experts,), role="vector", init="normal")]
+            specs.append(TensorSpec(p + n["router"], (self.num_experts, w)))
+            if self.has_correction:
+                specs.append(TensorSpec(p + n["correction"], (self.num_experts,), role="vector", init="normal"))
         if self.shared_size is not None:
             q, s = p + n["shared"], self.shared_size
             specs += [TensorSpec(q + n["gate"], (s, w)), TensorSpec(q + n["up"], (s, w)),
@@ -91,9 +101,9 @@ class RoutedExperts(FeedForward):
     def load(self, tensors):
         p, n = self.prefix, self.names
         names = [p + n["expert"].format(e) for e in range(self.num_experts)]
-        # [experts, 2F, W]: an expert's gate rows, then its up rows; [experts, W, F]
-        self.w_gate_up = torch.stack([torch.cat([tensors[q + n["gate"]], tensors[q + n["up"]]], dim=0)
-                                      for q in names]).contiguous()
+        # [experts, 2F, W]: an expert's gate rows, then its up rows (without a gate: [experts, F, W]); [experts, W, F]
+        self.w_gate_up = torch.stack([torch.cat([tensors[q + n[x]] for x in (("gate", "up") if self.gated else ("up",))],
+                                                dim=0) for q in names]).contiguous()
         self.w_down = torch.stack([tensors[q + n["down"]] for q in names]).contiguous()
         if self.shared_size is not None:
             q = p + n["shared"]
@@ -111,7 +121,8 @@ class RoutedExperts(FeedForward):
         if have % 8:
             rows.append(torch.zeros(8 - have % 8, self.hidden_size, dtype=rows[0].dtype, device=rows[0].device))
         self.w_router = torch.cat(rows, dim=0).contiguous()
-        self.correction = tensors[p + n["correction"]]
+        if self.has_correction:
+            self.correction = tensors[p + n["correction"]]
 
     def _shared(self, x):
         if self.shared_size is None:
@@ -125,11 +136,11 @@ class RoutedExperts(FeedForward):
         if self.score == "table":
             choice = ops.TableChoice(step.input_ids, self.table, self.route_scale / self.top)
             return ops.routed_experts(x, choice, None, self.w_gate_up, self.w_down, self._shared(x), None, -1,
-                                      self.out_dtype, limited=self.limited)
+                                      self.out_dtype, limited=self.limited, gated=self.gated)
         logits = ops.linear(x, self.w_router, out_dtype=torch.float32 if x.dtype != torch.float32 else None)
         ids, weights = ops.route_experts(logits, self.correction, self.num_experts, self.top, self.group_count,
                                          self.group_keep, self.route_scale, self.weight_eps, score=self.score,
                                          group_top=self.group_top, normalize=self.normalize)
         return ops.routed_experts(x, ids, weights, self.w_gate_up, self.w_down, self._shared(x), logits,
                                   self.num_experts if self.shared_gate else -1, self.out_dtype,
-                                  limited=self.limited)
+                                  limited=self.limited, gated=self.gated)

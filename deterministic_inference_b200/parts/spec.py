@@ -48,6 +48,8 @@ class ScheduleEntry:
     writes_cache: bool = True
     enter_vector: Optional[int] = None   # the plan's ``stream_addend`` adds its vector of this index
                                          # to the residual stream right before the layer runs
+    enters: bool = False                 # the plan's ``stream_entry`` replaces the residual stream right
+                                         # before the layer runs
 
 
 @dataclass(frozen=True)
@@ -64,12 +66,15 @@ class ModelPlan:
     ignored_names: tuple = ()         # checkpoint tensors that may be present and are not used
     ignored_substrings: tuple = ()
     stream_addend: Optional[PartSpec] = None   # learned vectors that schedule entries add to the stream
+    stream_entry: Optional[PartSpec] = None    # what schedule entries replace the stream by on entry
 
     def validate(self) -> None:
         writers: dict[int, int] = {}
         for pos, e in enumerate(self.schedule):
             if e.enter_vector is not None and self.stream_addend is None:
                 raise ValueError(f"schedule entry {pos} adds vector {e.enter_vector}, the plan has no stream addend")
+            if e.enters and self.stream_entry is None:
+                raise ValueError(f"schedule entry {pos} replaces the stream, the plan has no stream entry")
             if not 0 <= e.layer < len(self.layers):
                 raise ValueError(f"schedule entry {pos} names layer {e.layer}, "
                                  f"the plan has {len(self.layers)}")

@@ -131,7 +131,7 @@ def gather_rows(x, index):
     """sid/model/qwen3.py:113"""
     if hasattr(x, "eps") and hasattr(x, "weight"):       # a norm works row by row: gather first
         return type(x)(gather_rows(x.x, index), x.weight, x.eps)
-    if hasattr(x, "terms"):
+    if hasattr(x, "terms") or hasattr(x, "bias"):
         x = _plain(x)
     return x[index.long()].contiguous()
 
@@ -200,6 +200,8 @@ def _plain(x):
     """A float32 tensor of a weighted sum that is not added up yet, or of a tensor."""
     if hasattr(x, "eps") and hasattr(x, "weight"):       # a part's output under its post norm
         return _rms(_plain(x.x), x.weight, x.eps)
+    if hasattr(x, "bias"):                                # a projection whose bias is still to be added
+        return _plain(x.x) + x.bias
     if hasattr(x, "parts"):                               # split-k partial products
         total = x.parts[0].float().clone()
         for i in range(1, x.parts.shape[0]):
@@ -221,6 +223,26 @@ def stream_rms_norm(stream, weight, eps, out_dtype, add=None):
     if add is not None:
         stream += _plain(add)
     return _rms(stream, weight, eps).to(out_dtype)
+
+
+def stream_terms_(stream, term=None, norm=None, weight=None, eps=0.0, out=None):
+    if term is not None:
+        stream += _plain(term)
+    if out is not None:
+        y = stream
+        if norm == "rms":
+            y = _rms(stream, weight, eps)
+        elif norm == "layer":
+            y = stream - stream.mean(-1, keepdim=True)
+            y = y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) * weight
+        out.copy_(y.to(out.dtype))
+    return stream
+
+
+def stream_layer_norm(stream, weight, eps, out_dtype, add=None):
+    out = torch.empty(stream.shape, dtype=out_dtype)
+    stream_terms_(stream, add, "layer", weight, eps, out)
+    return out
 
 
 def xielu(z, alpha_p, alpha_n, out_dtype):
@@ -344,23 +366,23 @@ def limited_gate(gate_up, limit, alpha, out_dtype):
     return (g * torch.sigmoid(alpha * g) * (u + 1.0)).to(out_dtype)
 
 
-def _rotate_first(x, positions, freq, rot):
+def _rotate_first(x, positions, freq, rot, amp=1.0):
     """x [T, heads, D] float32: elements i and i + rot / 2 (i < rot / 2) turned by position * freq[i]."""
     if freq is None or rot == 0:
         return x
     half = rot // 2
     a = positions[:x.shape[0]].float()[:, None] * freq[None, :]
-    c, s = torch.cos(a)[:, None, :], torch.sin(a)[:, None, :]
+    c, s = amp * torch.cos(a)[:, None, :], amp * torch.sin(a)[:, None, :]
     u, v = x[..., :half], x[..., half:rot]
     return torch.cat([u * c - v * s, v * c + u * s, x[..., rot:]], dim=-1)
 
 
-def _rotate_pairs(x, positions, freq, rot):
+def _rotate_pairs(x, positions, freq, rot, amp=1.0):
     """x [T, heads, D] float32: elements 2i and 2i + 1 (i < rot / 2) turned by position * freq[i]."""
     if freq is None or rot == 0:
         return x
     a = positions[:x.shape[0]].float()[:, None] * freq[None, :]
-    c, s = torch.cos(a)[:, None, :], torch.sin(a)[:, None, :]
+    c, s = amp * torch.cos(a)[:, None, :], amp * torch.sin(a)[:, None, :]
     u, v = x[..., 0:rot:2], x[..., 1:rot:2]
     out = x.clone()
     out[..., 0:rot:2] = u * c - v * s
@@ -370,7 +392,7 @@ def _rotate_pairs(x, positions, freq, rot):
 
 def attn_prepare(proj, num_heads, num_kv_heads, head_dim, v_head_dim, q_norm_weight, k_norm_weight, eps, freq,
                  rotary_dim, positions, kv_cache, slot_mapping, page_size, out_dtype, bias=None, norm_scope="head",
-                 rotary_layout="halves", conv_weight=None, conv_state=None, step=None):
+                 rotary_layout="halves", conv_weight=None, conv_state=None, step=None, amplitude=1.0):
     t = proj.shape[0]
     nq, nk, nv = num_heads * head_dim, num_kv_heads * head_dim, num_kv_heads * v_head_dim
     x = _plain(proj)[:, :nq + nk + nv]
@@ -391,7 +413,7 @@ def attn_prepare(proj, num_heads, num_kv_heads, head_dim, v_head_dim, q_norm_wei
     q, k = q.reshape(t, num_heads, head_dim), k.reshape(t, num_kv_heads, head_dim)
     v = x[:, nq + nk:nq + nk + nv].reshape(t, num_kv_heads, v_head_dim)
     rotate = _rotate_pairs if rotary_layout == "pairs" else _rotate_first
-    q, k = rotate(q, positions, freq, rotary_dim), rotate(k, positions, freq, rotary_dim)
+    q, k = rotate(q, positions, freq, rotary_dim, amplitude), rotate(k, positions, freq, rotary_dim, amplitude)
     if kv_cache is not None:
         flat = kv_cache.view(kv_cache.shape[0], -1)
         v_base = num_kv_heads * page_size * head_dim
@@ -426,13 +448,36 @@ def latent_prepare(proj, num_heads, plain_dim, rot_dim, rank, latent_norm_weight
     return q
 
 
+def latent_rows(proj, q_col, q_rank, q_norm_weight, kv_col, rank, rot_dim, latent_norm_weight, eps, freq, positions,
+                kv_cache, slot_mapping, page_size, out_dtype, rotary_layout="halves", amplitude=1.0):
+    x = _plain(proj).to(out_dtype).float()
+    t = x.shape[0]
+    if kv_cache is not None:
+        row = _rms(x[:, kv_col:kv_col + rank], latent_norm_weight, eps)
+        if rot_dim:
+            turn = _rotate_pairs if rotary_layout == "pairs" else _rotate_first
+            key = x[:, None, kv_col + rank:kv_col + rank + rot_dim]
+            row = torch.cat([row, turn(key, positions, freq, rot_dim, amplitude)[:, 0]], dim=-1)
+        rows = kv_cache.view(-1, rank + rot_dim)
+        for i, slot in enumerate(slot_mapping.tolist()[:t]):
+            if slot >= 0:
+                rows[slot] = row[i].to(out_dtype)
+    return _rms(x[:, q_col:q_col + q_rank], q_norm_weight, eps).to(out_dtype)
+
+
+def sigmoid_gate_(x, gate, gate_col, per=1):
+    g = _plain(gate).to(x.dtype).float()[:, gate_col:gate_col + x.shape[1] // per]
+    x.copy_((x.float() * torch.sigmoid(g.repeat_interleave(per, dim=1))).to(x.dtype))
+    return x
+
+
 def heads_linear(x, weight, out):
     out.copy_(torch.einsum("mhk,hkn->mhn", x.float(), weight.float()).to(out.dtype))
     return out
 
 
 def masked_attention(q, kv_cache, meta, scale, num_kv_heads, v_head_dim, page_size, mask="causal", mask_size=None,
-                     sink=None, gate=None, gate_col=0, values_in_keys=False, keep_first=0, softcap=None):
+                     sink=None, gate=None, gate_col=0, values_in_keys=False, keep_first=0, softcap=None, gate_per_head=False):
     t, hq, dk = q.shape
     flat = kv_cache.view(kv_cache.shape[0], -1)
     keys_of = flat[:, :num_kv_heads * page_size * dk].view(-1, num_kv_heads, page_size, dk)
@@ -460,7 +505,9 @@ def masked_attention(q, kv_cache, meta, scale, num_kv_heads, v_head_dim, page_si
             w = torch.softmax(s, dim=0)[:js.shape[0]]
             out[i, h] = w @ v
     out = out.to(q.dtype)
-    if g_all is not None:
+    if g_all is not None and gate_per_head:
+        out = (out.float() * torch.sigmoid(g_all[:, gate_col:gate_col + hq])[:, :, None]).to(q.dtype)
+    elif g_all is not None:
         cols = g_all[:, gate_col:gate_col + hq * v_head_dim].reshape(t, hq, v_head_dim)
         out = (out.float() * torch.sigmoid(cols)).to(q.dtype)
     return out
@@ -579,8 +626,8 @@ def state_space(proj, conv_weight, conv_bias, a_log, dt_bias, d_skip, norm_weigh
 def route_experts(logits, correction, num_experts, top, group_count, group_keep, scale, eps, score="sigmoid",
                   group_top=2, normalize=True):
     z = _plain(logits)[:, :num_experts]
-    s = torch.softmax(z, dim=-1) if score == "softmax" else torch.sigmoid(z)
-    choice = s + correction
+    s = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z, dim=-1)
+    choice = (z if score == "chosen_softmax" else s) + (0.0 if correction is None else correction)
     per = num_experts // group_count
     by_group = choice.view(-1, group_count, per)
     group_score = by_group.topk(min(group_top, per), dim=-1).values.sum(-1)
@@ -624,7 +671,30 @@ def retention(proj, decay, freq, state, step, num_heads, head_dim, v_head_dim, n
     return (o * (g * torch.sigmoid(g))).to(out_dtype)
 
 
-def routed_experts(x, ids, weights, w_gate_up, w_down, shared, logits, shared_gate_col, out_dtype, limited=None):
+def gated_linear_attention(proj, hidden, hidden_col, a2_t, a2_bias, tau, norm_weight, state, step, num_heads, head_dim,
+                           v_head_dim, norm_eps, out_dtype):
+    h, d, e = num_heads, head_dim, v_head_dim
+    z = _plain(hidden)[:, hidden_col:hidden_col + a2_t.shape[0]] @ a2_t.float() + a2_bias
+    x = _plain(proj).to(out_dtype).float()
+    t = x.shape[0]
+    alpha = torch.exp(torch.nn.functional.logsigmoid(z) / tau).reshape(t, h, d)
+    q, k = x[:, :h * d].reshape(t, h, d) * d ** -0.5, x[:, h * d:2 * h * d].reshape(t, h, d)
+    v, g = x[:, 2 * h * d:2 * h * d + h * e].reshape(t, h, e), x[:, 2 * h * d + h * e:2 * h * (d + e)]
+    cu, slots = step.cu_q_lens.tolist(), step.state_slots.tolist()
+    o = torch.zeros(t, h, e)
+    for b in range(len(slots)):
+        s = state[slots[b]].view(h, d, e).clone() if slots[b] else torch.zeros(h, d, e)
+        for i in range(cu[b], cu[b + 1]):
+            s = alpha[i][:, :, None] * s + k[i][:, :, None] * v[i][:, None, :]
+            o[i] = torch.einsum("hde,hd->he", s, q[i])
+        if slots[b]:
+            state[slots[b]] = s.reshape(-1)
+    o = (o / torch.sqrt(o.square().mean(-1, keepdim=True) + norm_eps) * norm_weight).reshape(t, h * e)
+    return (o * (g * torch.sigmoid(g))).to(out_dtype)
+
+
+def routed_experts(x, ids, weights, w_gate_up, w_down, shared, logits, shared_gate_col, out_dtype, limited=None,
+                   gated=True):
     t, w = x.shape
     if hasattr(ids, "table"):               # a table's choice by token id
         weight, ids = ids.weight, ids.table[ids.token_ids.long()[:t]]
@@ -635,7 +705,9 @@ def routed_experts(x, ids, weights, w_gate_up, w_down, shared, logits, shared_ga
         for j in range(ids.shape[1]):
             e = int(ids[i, j])
             gu = w_gate_up[e].float() @ x[i].float()
-            if limited is None:
+            if not gated:
+                hdn = 0.5 * gu * (1.0 + torch.erf(gu * 0.5 ** 0.5))
+            elif limited is None:
                 hdn = gu[:f] * torch.sigmoid(gu[:f]) * gu[f:]
             else:
                 a, b = gu[:f].clamp(max=limited[0]), gu[f:].clamp(-limited[0], limited[0])
@@ -649,7 +721,7 @@ def routed_experts(x, ids, weights, w_gate_up, w_down, shared, logits, shared_ga
     return out
 
 
-ALL = ("retention", "squared_relu", "squared_relu_linear", "state_space", "scale_", "stream_read", "gated_delta_rule", "gated_linear_recurrence", "route_experts", "routed_experts",
+ALL = ("stream_terms_", "stream_layer_norm", "latent_rows", "sigmoid_gate_", "gated_linear_attention", "retention", "squared_relu", "squared_relu_linear", "state_space", "scale_", "stream_read", "gated_delta_rule", "gated_linear_recurrence", "route_experts", "routed_experts",
        "embedding_scaled", "stream_add_", "limited_gate", "attn_prepare", "latent_prepare", "heads_linear",
        "masked_attention", "embedding_positions", "stream_rms_norm", "xielu", "softcap_", "qkv_bias_cache", "sigmoid_attention",
        "delta_rule", "patch_token_ids", "embedding", "rms_norm", "add_rms_norm", "qk_norm_rope_cache", "reshape_and_cache",
