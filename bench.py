@@ -651,10 +651,8 @@ def design_arm(a) -> int:
                         2 * (2 * t * hq * d + batch * hkv * 2 * d * held), 4 * keys * hq * d)
                     proj = torch.randn(t, (2 * hq + 2 * hkv) * d, device=dev)
                     o = torch.randn(t, hq * d, device=dev).to(bf)
-                    from ctypes import c_int, c_longlong
-                    row(f"{what}: sigmoid gate on the heads", timed(lambda: ops._check(ops._lib("masked_attention").dib_sigmoid_gate_(
-                        ops._ptr(o), *ops._source_args(proj), c_longlong(proj.shape[1]), c_longlong((hq + 2 * hkv) * d),
-                        c_int(t), c_int(hq * d), c_int(1), ops._stream()), "gate")), t * hq * d * (2 + 2 + 4), 0)
+                    row(f"{what}: sigmoid gate on the heads", timed(lambda: ops.sigmoid_gate_(o, proj, (hq + 2 * hkv) * d)),
+                        t * hq * d * (2 + 2 + 4), 0)
                     freq = runner.model.mixers[0].freq
                     row(f"{what}: q/k norm + partial rotation + cache write", timed(lambda: ops.attn_prepare(
                         proj, hq, hkv, d, d, one_w[:d].contiguous(), one_w[:d].contiguous(), 1e-6, freq, d // 2,

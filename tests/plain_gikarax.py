@@ -256,8 +256,8 @@ def expert(h, w, p, rnd=_keep):
     return rnd(rnd(gelu(rnd(h @ w[p + "up"].T))) @ w[p + "down"].T)
 
 
-def mixture(h, w, p, c, rnd=_keep, choose=chosen_experts):
-    ids, weights = choose(h, w, p, c["router"]["top"])
+def mixture(h, w, p, c, rnd=_keep, choose=None):
+    ids, weights = (choose or chosen_experts)(h, w, p, c["router"]["top"])
     out = torch.zeros_like(h)
     for e in range(c["router"]["experts"]):
         share = (weights * (ids == e)).sum(-1)
@@ -281,7 +281,7 @@ def layer_runs(cfg):
     return runs + [(i, False) for i in range(stop, n)]
 
 
-def forward(cfg, w, tokens, rnd=_keep, layers_out=None, choose=chosen_experts):
+def forward(cfg, w, tokens, rnd=_keep, layers_out=None, choose=None):
     """Logits [n, vocab] of one sequence.  ``layers_out``: a list that receives the residual stream
     after every layer run."""
     eps = float(cfg["norm"]["eps"])
