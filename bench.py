@@ -441,8 +441,46 @@ def nedupel_like(q, layers: int, rank: int, rot: int, r_heads: int, r_dim: int, 
         "layers": entries})
 
 
+GIKARAX_SIZES = {
+    # name -> the Gikarax sizes that go with the Qwen3 preset of DESIGN_SIZES[name]: the attention heads are
+    # Qwen3's, the gated linear attention is as wide as the model in heads of 128, the latents are 256 wide, and
+    # a token's experts hold as many weights as Bovitar's (the chosen ones and the shared one)
+    "0_6b": dict(window=1024, softcap=30.0, kv_rank=256, q_rank=512, r_heads=8, r_dim=128, decay_rank=16, experts=16,
+                 top=2, expert_ff=2304),
+    "8b": dict(window=4096, softcap=30.0, kv_rank=256, q_rank=1536, r_heads=32, r_dim=128, decay_rank=16, experts=32,
+               top=4, expert_ff=4608),
+}
+
+
+def gikarax_like(q, layers: int, window: int, softcap: float, kv_rank: int, q_rank: int, r_heads: int, r_dim: int,
+                 decay_rank: int, experts: int, top: int, expert_ff: int):
+    """A Gikarax configuration with the layer sizes of the Qwen3 configuration ``q`` and ``layers`` (at least 4)
+    layer runs: windowed attention, parallel and latent layers in turn, the parallel one behind the first
+    layer run twice in a row."""
+    from deterministic_inference_b200.config.gikarax_config import GikaraxConfig
+    d = q.head_dim
+    heads = {"heads": q.num_attention_heads, "kv_heads": q.num_key_value_heads, "dim": d, "vdim": d, "scale": d ** -0.5}
+    mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}}
+    attention = {"type": "attention", "mlp": mlp, "mixer": dict(
+        heads, softcap=softcap, mask={"size": window},
+        rot={"base": 500000.0, "dims": d // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}})}
+    par = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": dict(heads, rot={"base": 500000.0, "dims": d // 2,
+                                 "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}),
+        "right": {"heads": r_heads, "dim": r_dim, "vdim": r_dim, "tau": 16.0, "decay_rank": decay_rank}}}
+    latent = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": q.num_attention_heads, "dim": d, "vdim": d, "kv_rank": kv_rank, "q_rank": q_rank, "scale": d ** -0.5}}
+    return GikaraxConfig.from_dict({
+        "architecture": "Gikarax", "vocab": q.vocab_size, "width": q.hidden_size, "max_positions": 8192,
+        "norm": {"eps": 1e-6}, "loop": {"start": 1, "stop": 2, "times": 2},
+        "layers": [(attention, par, latent)[i % 3] for i in range(layers - 1)]})
+
+
 def design_arm(a) -> int:
-    """``--design nedupel``: the Nedupel design beside Zatirax (the closest: latent attention, a float32
+    """``--design gikarax``: the Gikarax design beside Bovitar (the closest: attention beside a recurrence with
+    both branches normed, capped scores, routed experts, a float32 stream), its kernels also beside Nedupel's
+    retention and Zatirax's latent rows.
+    ``--design nedupel``: the Nedupel design beside Zatirax (the closest: latent attention, a float32
     stream), its kernels also beside the state-space recurrence and the routed experts of the other designs.
     ``--design zatirax``: the same for the Zatirax design; ``--design kipezen``: for the Kipezen design,
     beside Gamilorn (the closest design) instead of Qwen3.  ``--design gamilorn``: prompt and decode throughput of the Gamilorn design at layer sizes of
@@ -1028,6 +1066,169 @@ def design_arm(a) -> int:
                     cache.release_slot(sl)
         return rows
 
+    def gikarax_kernel_rows(eng_g, eng_b, gcfg, bcfg):
+        """Gikarax's kernels on one layer's shapes and the like kernels of the other designs at equal sizes:
+        Bovitar's attention, branches' norm, state-space branch and feed-forward, Nedupel's retention with
+        the same heads and states, Zatirax's latent rows with the same widths.  A prompt of ``n_prompt`` tokens,
+        and a decode step of 8 requests with ``ctx`` cached tokens."""
+        rows = {}
+        hbm, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+        att, par, lat = (gcfg.layers[i]["mixer"] for i in range(3))
+        hq, hkv, d, w, win = att["heads"], att["kv_heads"], att["dim"], gcfg.width, att["mask"]["size"]
+        rh, rn, rp, rank = (par["right"][k] for k in ("heads", "dim", "vdim", "decay_rank"))
+        lh, ld, le, lc, lq = (lat[k] for k in ("heads", "dim", "vdim", "kv_rank", "q_rank"))
+        moe, b_par, b_mlp = gcfg.layers[0]["mlp"], bcfg.layers[1]["mixer"], bcfg.layers[0]["mlp"]
+        n_exp, top, eff = moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"]
+        bf = torch.bfloat16
+
+        def row(name, ms, nbytes, flops):
+            floor = max(nbytes / hbm, flops / tf) * 1e3
+            rows[name] = {"ms": round(ms, 4), "roofline_ms": round(floor, 4), "of_roofline": round(floor / ms, 4)}
+
+        for what, batch, q_len, before in (("prompt", 1, n_prompt, 0), ("decode_b8", 8, 1, ctx)):
+            t = batch * q_len
+            span = range(before, before + q_len)
+            x = torch.randn(t, w, device=dev).to(bf)
+            y = torch.randn(t, w, device=dev)
+            stream = torch.randn(t, w, device=dev)
+            one_w, one_d = torch.ones(w, device=dev), torch.ones(d, device=dev)
+            q = torch.randn(t, hq, d, device=dev).to(bf)
+            proj = torch.randn(t, (hq + 2 * hkv) * d + hq, device=dev)
+            for eng, mine in ((eng_g, True), (eng_b, False)):
+                runner, cache = eng.runner, eng.cache
+                slots = [cache.allocate_slot() for _ in range(batch)]
+                if before:
+                    for sl in slots:
+                        runner.step([SequenceInput(sl, prompt_of(1000, before), 0, [])])
+                entries = [SequenceInput(sl, [1] * q_len, before, []) for sl in slots]
+                for e_ in entries:
+                    cache.allocate(e_.slot, before + q_len)
+                cache.reset_fresh_state()
+                step = build_step_batch(entries, cache, dev)
+                blocks = runner.model.blocks
+
+                def attention_row(name, kv, seen, **kw):
+                    keys, held = batch * sum(seen(p) for p in span), seen(before + q_len - 1)
+                    row(f"{what}: {name}", timed(lambda: ops.masked_attention(
+                        q, kv.kv, kv.attention_meta, d ** -0.5, hkv, d, kv.page_size, **kw)),
+                        2 * (2 * t * hq * d + batch * hkv * 2 * d * held), 4 * keys * hq * d)
+                if not mine:
+                    pview, ssm, right = cache.view(1, step), blocks[1].mixer.branches[1], b_par["right"]
+                    kv, tail = pview.members[0].members[0], pview.members[0].members[1].state
+                    b_att = blocks[1].mixer.branches[0]
+                    attention_row("bovitar attention, causal, capped scores", kv, lambda p: p + 1,
+                                  softcap=b_par["left"]["softcap"])
+                    bproj = torch.randn(t, (hq + 2 * hkv) * d, device=dev)
+                    row(f"{what}: bovitar q/k/v convolutions + norm over the projection + rotation + cache write", timed(
+                        lambda: ops.attn_prepare(bproj, hq, hkv, d, d, b_att.q_norm, b_att.k_norm, 1e-6, b_att.freq,
+                                                 b_att.rotary_dim, step.positions, kv.kv, kv.slot_mapping, kv.page_size, bf,
+                                                 norm_scope="projection", conv_weight=b_att.conv, conv_state=tail, step=step)),
+                        bproj.numel() * 6 + batch * tail.shape[1] * 8, 0)
+                    sh, sp, sn, sg = right["heads"], right["vdim"], right["state"], right["groups"]
+                    sproj = torch.randn(t, ssm.w_in.shape[0], device=dev)
+                    row(f"{what}: bovitar state-space branch (convolution, recurrence, gated norm)", timed(
+                        lambda: ops.state_space(sproj, ssm.conv, ssm.conv_bias, ssm.a_log, ssm.dt_bias, ssm.d_skip,
+                                                ssm.norm_weight, pview.members[1].state, step, sh, sp, sn, sg,
+                                                right["norm_groups"], right["conv"], 1e-6, bf)),
+                        batch * sh * sn * sp * 8 + t * (sproj.shape[1] * 4 + sh * sp * 2), 5 * t * sh * sn * sp)
+                    row(f"{what}: bovitar two normed branches + add + norm of the float32 stream", timed(
+                        lambda: ops.stream_rms_norm(stream, one_w, 1e-6, bf, add=ops.WeightedSum(
+                            [(0.5, ops.NormedTerm(x, one_w, 1e-6)), (0.5, ops.NormedTerm(x, one_w, 1e-6))]))), t * w * 14, 0)
+                    ff = blocks[0].feed_forward
+                    b_exp, b_top = b_mlp["router"]["experts"], b_mlp["router"]["top"]
+                    b_eff, b_sff = b_mlp["expert"]["ff"], b_mlp["shared"]["ff"]
+                    row(f"{what}: bovitar feed-forward (router, shared expert, routed experts)", timed(lambda: ff.forward(x)),
+                        (min(b_exp, t * b_top) * b_eff + b_sff) * 3 * w * 2 + t * w * 6, 6 * t * (b_top * b_eff + b_sff) * w)
+                    # the experts alone, the same choice and as many weights (gated experts of two thirds the width)
+                    ids, share = ops.route_experts(torch.randn(t, n_exp, device=dev), None, n_exp, top, 1, 1, 1.0, 0.0,
+                                                   score="chosen_softmax")
+                    gf = eff * 2 // 3
+                    gu = torch.randn(n_exp, 2 * gf, w, device=dev).to(bf)
+                    dn = torch.randn(n_exp, w, gf, device=dev).to(bf)
+                    row(f"{what}: gated experts (Kipezen's, Bovitar's) of as many weights, the same choice", timed(
+                        lambda: ops.routed_experts(x, ids, share, gu, dn, None, None, -1, bf)),
+                        min(n_exp, t * top) * gf * 3 * w * 2 + t * w * 6, 6 * t * top * gf * w)
+                    for sl in slots:
+                        cache.release_slot(sl)
+                    continue
+                view, pview, lview = cache.view(0, step), cache.view(1, step), cache.view(3, step)
+                a_mix, l_half, gla, l_mix = blocks[0].mixer, *blocks[1].mixer.branches, blocks[2].mixer
+                attention_row("attention, window, capped scores, sink, a gate per head", view, lambda p: min(p + 1, win),
+                              mask="window", mask_size=win, sink=a_mix.sinks, softcap=att["softcap"], gate=proj,
+                              gate_col=(hq + 2 * hkv) * d, gate_per_head=True)
+                attention_row("the left half's attention, causal", pview.members[0], lambda p: p + 1)
+                row(f"{what}: q/k norm + stretched rotation + cache write", timed(lambda: ops.attn_prepare(
+                    proj, hq, hkv, d, d, one_d, one_d, 1e-6, a_mix.freq, a_mix.rotary_dim, step.positions, view.kv,
+                    view.slot_mapping, view.page_size, bf)), proj.numel() * 6, 0)
+                lkv = pview.members[0]
+                row(f"{what}: q/k/v bias + blended rotation + cache write", timed(lambda: ops.attn_prepare(
+                    proj, hq, hkv, d, d, None, None, 0.0, l_half.freq, l_half.rotary_dim, step.positions, lkv.kv,
+                    lkv.slot_mapping, lkv.page_size, bf, bias=l_half.b_in, amplitude=l_half.amplitude)), proj.numel() * 6, 0)
+                state = pview.members[1].state
+                gproj, hid = torch.randn(t, 2 * rh * (rn + rp), device=dev).to(bf), torch.randn(t, rank, device=dev)
+                rec_bytes, rec_flops = gproj.numel() * 2 + t * rh * rp * 2 + batch * rh * rn * rp * 8, 4 * t * rh * rn * rp
+                row(f"{what}: gated linear attention (decays, recurrence, norm, gate)", timed(
+                    lambda: ops.gated_linear_attention(gproj, hid, 0, gla.a2_t, gla.a2_bias, 16.0, gla.norm_weight, state, step,
+                                                       rh, rn, rp, 1e-6, bf)), rec_bytes + t * (rank * 4), rec_flops)
+                decay, turn = torch.full((rh,), 0.99, device=dev), torch.full((rn // 2,), 0.1, device=dev)
+                row(f"{what}: retention (Nedupel's) of the same heads and states", timed(lambda: ops.retention(
+                    gproj, decay, turn, state, step, rh, rn, rp, 1e-6, bf)), rec_bytes, rec_flops)
+
+                ql = torch.randn(t, lh, lc, device=dev).to(bf)
+                keys, held = batch * sum(p + 1 for p in span), before + q_len
+                row(f"{what}: latent attention, causal", timed(lambda: ops.masked_attention(
+                    ql, lview.kv, lview.attention_meta, ld ** -0.5, 1, lc, lview.page_size, values_in_keys=True)),
+                    2 * (2 * t * lh * lc + batch * lc * held), 4 * keys * lh * lc)
+                row(f"{what}: the same with a rotated part of 64 (Zatirax's, Nedupel's)", timed(lambda: ops.masked_attention(
+                    ql, lview.kv, lview.attention_meta, ld ** -0.5, 1, lc - 64, lview.page_size, values_in_keys=True)),
+                    2 * (t * lh * (2 * lc - 64) + batch * lc * held), 2 * keys * lh * (2 * lc - 64))
+                lproj = torch.randn(t, lq + lc + lh * le, device=dev).to(bf)
+                lkw = dict(positions=step.positions, kv_cache=lview.kv, slot_mapping=lview.slot_mapping,
+                           page_size=lview.page_size, out_dtype=bf)
+
+                def latent_side():
+                    c_q = ops.latent_rows(lproj, 0, lq, l_mix.q_norm, lq, lc, 0, l_mix.latent_norm, 1e-6, None, **lkw)
+                    heads = ops.as_tensor(ops.linear(c_q, l_mix.w_q_up))
+                    qq = torch.empty(t, lh, lc, dtype=bf, device=dev)
+                    ops.heads_linear(heads.view(t, lh, ld), l_mix.w_key, qq)
+                    oo = torch.empty(t, lh, le, dtype=bf, device=dev)
+                    ops.heads_linear(ql, l_mix.w_value, oo)
+                    ops.sigmoid_gate_(oo.view(t, lh * le), lproj, lq + lc)
+                row(f"{what}: latent rows + query map + the two products per head + gate", timed(latent_side),
+                    2 * (lproj.numel() + t * lh * (2 * lc + 2 * ld + 3 * le) + lh * lc * (ld + le) + lq * lh * ld),
+                    2 * t * lh * (lc * (ld + le) + lq * ld))
+                zd, zc = ld - 64, lc - 64
+                zproj = torch.randn(t, lh * ld + lc, device=dev).to(bf)
+                wk, wv = torch.randn(lh, zd, zc, device=dev).to(bf), torch.randn(lh, zc, le, device=dev).to(bf)
+                zfreq, znorm = torch.full((32,), 0.1, device=dev), torch.ones(zc, device=dev)
+
+                def zatirax_side():
+                    qq = ops.latent_prepare(zproj, lh, zd, 64, zc, znorm, 1e-6, zfreq, **lkw)
+                    ops.heads_linear(zproj.as_strided((t, lh, zd), (zproj.shape[1], ld, 1)), wk, qq[:, :, :zc])
+                    oo = torch.empty(t, lh, le, dtype=bf, device=dev)
+                    ops.heads_linear(ql[:, :, :zc], wv, oo)
+                row(f"{what}: latent rows + the two products per head (Zatirax's)", timed(zatirax_side),
+                    2 * (zproj.numel() + t * lh * (2 * zc + 64 + le) + lh * zc * (zd + le)), 2 * t * lh * zc * (zd + le))
+                branches = [(0.5, ops.NormedTerm(ops.BiasedTerm(x, one_w), one_w, 1e-6)), (0.5, ops.NormedTerm(x, one_w, 1e-6)),
+                            (1.0, y)]
+                row(f"{what}: two normed branches + feed-forward + add + layer norm of the float32 stream", timed(
+                    lambda: ops.stream_layer_norm(stream, one_w, 1e-6, bf, add=ops.WeightedSum(branches))), t * w * 18, 0)
+                ent = runner.model.stream_entry
+                kept = ent.start(stream)
+                row(f"{what}: a pass's entry (stream read, product, copy of the start's share)", timed(
+                    lambda: ent.enter(y, stream, kept, False)), t * w * (4 * 3 + 2 * 2 + 4 + 8) + 2 * w * w, 2 * t * w * w)
+                ff = blocks[0].feed_forward
+                row(f"{what}: feed-forward (router, experts without a gate)", timed(lambda: ff.forward(x)),
+                    min(n_exp, t * top) * eff * 2 * w * 2 + t * w * 6, 4 * t * top * eff * w)
+                ids, share = ops.route_experts(torch.randn(t, n_exp, device=dev), None, n_exp, top, 1, 1, 1.0, 0.0,
+                                               score="chosen_softmax")
+                row(f"{what}: experts without a gate", timed(lambda: ops.routed_experts(
+                    x, ids, share, ff.w_gate_up, ff.w_down, None, None, -1, bf, gated=False)),
+                    min(n_exp, t * top) * eff * 2 * w * 2 + t * w * 6, 4 * t * top * eff * w)
+                for sl in slots:
+                    cache.release_slot(sl)
+        return rows
+
     sampler = ClockSampler()
     sampler.start()
     sizes = {}
@@ -1048,6 +1249,11 @@ def design_arm(a) -> int:
             beside, bcfg = "zatirax", zatirax_like(qcfg, n_layers, **ZATIRAX_SIZES[name])
             extra = NEDUPEL_SIZES[name]
             gcfg = nedupel_like(qcfg, n_layers, **extra)
+        elif a.design == "gikarax":
+            # beside Bovitar, the closest design, at the same layer sizes
+            beside, bcfg = "bovitar", bovitar_like(qcfg, n_layers, **BOVITAR_SIZES[name])
+            extra = GIKARAX_SIZES[name]
+            gcfg = gikarax_like(qcfg, n_layers, **extra)
         elif a.design == "bovitar":
             # beside Kipezen, the closest design, at the same layer sizes
             beside, bcfg = "kipezen", kipezen_like(qcfg, n_layers, **KIPEZEN_SIZES[name])
@@ -1069,14 +1275,15 @@ def design_arm(a) -> int:
                 r[f"decode_b{b}_tok_s"] = round(b / (dms / 1e3))
             out[label + "_result"] = r
         rows_of = {"zatirax": zatirax_kernel_rows, "kipezen": kipezen_kernel_rows,
-                   "bovitar": bovitar_kernel_rows, "nedupel": nedupel_kernel_rows}.get(a.design, kernel_rows)
+                   "bovitar": bovitar_kernel_rows, "nedupel": nedupel_kernel_rows,
+                   "gikarax": gikarax_kernel_rows}.get(a.design, kernel_rows)
         out["kernels"] = rows_of(engines[a.design], engines[beside], gcfg, bcfg)
         sizes[name] = out
         del engines
         import gc
         gc.collect()
         torch.cuda.empty_cache()
-    beside = {"kipezen": "gamilorn", "bovitar": "kipezen", "nedupel": "zatirax"}.get(a.design, "qwen3")
+    beside = {"kipezen": "gamilorn", "bovitar": "kipezen", "nedupel": "zatirax", "gikarax": "bovitar"}.get(a.design, "qwen3")
     print(json.dumps({"metric": f"{a.design} beside {beside} at equal layer sizes (bf16, 1 B200)", "impl": "ours",
                       "dtype": "bf16", "data": "synthetic, random weights", "n_gpus": 1,
                       "prompt_tokens": n_prompt, "decode_context": ctx, "decode_steps": a.point_steps,
@@ -1111,8 +1318,8 @@ def main() -> int:
     ap.add_argument("--profile", default=None, choices=["decode", "prefill"],
                     help="bracket this region with cudaProfilerStart/Stop (for ncu "
                          "--profile-from-start off); the numbers of such a run are not a result")
-    ap.add_argument("--design", default=None, choices=["gamilorn", "zatirax", "kipezen", "bovitar", "nedupel"],
-                    help="measure this design beside Qwen3 (kipezen: beside Gamilorn; bovitar: beside Kipezen; nedupel: beside Zatirax) at equal layer sizes instead of the default "
+    ap.add_argument("--design", default=None, choices=["gamilorn", "zatirax", "kipezen", "bovitar", "nedupel", "gikarax"],
+                    help="measure this design beside Qwen3 (kipezen: beside Gamilorn; bovitar: beside Kipezen; nedupel: beside Zatirax; gikarax: beside Bovitar) at equal layer sizes instead of the default "
                          "workload (prints a line of its own)")
     ap.add_argument("--design-sizes", default="0_6b,8b", help=f"of {sorted(DESIGN_SIZES)}")
     ap.add_argument("--design-layers", type=int, default=4)

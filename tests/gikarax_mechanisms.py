@@ -144,6 +144,9 @@ def window_case(tmp, dtype, device, heads, kv_heads, dim, vdim, window, rot, pag
         direction = torch.ones(dim)
         if 0 < rot < dim:
             direction[:rot] = 0.0                 # where it can, outside the rotated part
+        elif rot:
+            direction = torch.zeros(dim)          # else on the pairs that turn slowest
+            direction[rot // 2 - 2:rot // 2] = math.sqrt(dim / 2.0)
         t["l0.mix.k"][:, 0] = direction.repeat(kv_heads)
         t["l0.mix.q"][:, 1] = direction.repeat(heads)
         t["l0.mix.k"].mul_(0.7)
@@ -354,9 +357,9 @@ def latent_case(tmp, dtype, device, heads, dim, vdim, kv_rank, q_rank, page, n=3
         t[p + "dq"].mul_(0.3)
         t[p + "dq"][0, 1] = 1.5
         t[p + "uk"].mul_(0.2)
-        t[p + "uk"][:, 0] = 1.0
+        t[p + "uk"][:, 0] = math.sqrt(24.0 / kv_rank)      # (an element of a normed latent grows with its size)
         t[p + "uq"].mul_(0.3)
-        t[p + "uq"][:, 0] = 0.6
+        t[p + "uq"][:, 0] = 0.6 * math.sqrt(12.0 / q_rank)
 
     d = gu.write_model(config, seed, tmp, edit)
     toks = filler_tokens(97, n, seed)
