@@ -3,8 +3,8 @@
 // proj row (row_width elements): [q: H N | k: H N | v: H P | g: H P | anything].  Per head, with a state S
 // [N][P] from zero and a decay alpha per (token, row of S):
 //     S <- diag(alpha) S + k v^T;     o = S^T (q q_scale);     out = o / sqrt(mean(o^2) + eps) * w * silu(g),
-// w [P] shared by the heads.  gla_decay_kernel leaves log alpha = log(sigmoid(z)) / tau, z = hidden A2^T + b,
-// as float32 [T][H N].  A request's state slot holds the heads' states [H][N][P], float32; slot 0 is no
+// w [P] shared by the heads, log alpha = log(sigmoid(z)) / tau with z = hidden A2^T + b, `hidden` R float32
+// numbers a token; both forms make the decays they need from it.  A request's state slot holds the heads' states [H][N][P], float32; slot 0 is no
 // request's: a sequence on it starts from zeros and stores nothing.
 //
 // Two forms.
@@ -50,38 +50,20 @@ constexpr float LEAST = -9.0f;         // the smallest log decay of the chunked 
 constexpr int RUN = 16;                // tokens of a run
 constexpr int RUNS = CH / RUN;
 
-// ---- decays ------------------------------------------------------------------------------------------
-// grid (ceil(C / 256), ceil(T / GD)); a thread per channel, GD tokens; k in ascending order.
-constexpr int GD = 8;
-template <typename T>
-__global__ void __launch_bounds__(256)
-gla_decay_kernel(Source hidden, long long row_width, long long at, const T* __restrict__ a2_t,
-                 const float* __restrict__ bias, float tau, float* out, int T_tokens, int R, int C) {
-  extern __shared__ float hs[];        // [GD][R]
-  pdl_prologue(hidden.p);
-  const int t0 = blockIdx.y * GD, c = blockIdx.x * 256 + threadIdx.x;
-  for (int i = threadIdx.x; i < GD * R; i += 256) {
-    const int j = i / R, r = i - j * R;
-    hs[i] = t0 + j < T_tokens ? source_load(hidden, (long long)(t0 + j) * row_width + at + r) : 0.f;
-  }
-  __syncthreads();
-  if (c >= C) return;
-  float acc[GD];
-#pragma unroll
-  for (int j = 0; j < GD; ++j) acc[j] = 0.f;
-#pragma unroll 4
-  for (int r = 0; r < R; ++r) {
-    const float w = Elem<T>::load(a2_t + (long long)r * C + c);
-#pragma unroll
-    for (int j = 0; j < GD; ++j) acc[j] = __fmaf_rn(hs[j * R + r], w, acc[j]);
-  }
-  const float b = bias[c];
-#pragma unroll
-  for (int j = 0; j < GD; ++j)
-    if (t0 + j < T_tokens) {
-      const float z = __fadd_rn(acc[j], b);
-      out[(long long)(t0 + j) * C + c] = (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) / tau;
-    }
+// What the decays are made of: R numbers a token at column `at` of rows row_width apart, the map a2_t [R][H N]
+// (dtype 0 float32, 1 bfloat16) and its bias.
+struct Decays {
+  Source hidden;
+  long long row_width, at;
+  const void* a2_t;
+  int dtype;
+  const float* bias;
+  float tau;
+  int R;
+};
+__device__ __forceinline__ float log_decay(float sum, float bias, float tau) {
+  const float z = __fadd_rn(sum, bias);
+  return (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) / tau;
 }
 
 // ---- token by token --------------------------------------------------------------------------------
@@ -93,13 +75,13 @@ gla_decay_kernel(Source hidden, long long row_width, long long at, const T* __re
 constexpr int ST = 256;
 template <int VEC>
 __global__ void __launch_bounds__(ST)
-gla_step_kernel(Source proj, long long row_width, const float* log_decay, float* state, long long slot_stride,
+gla_step_kernel(Source proj, long long row_width, Decays dec, float* state, long long slot_stride,
                 const int* __restrict__ cu_q_lens, const int* __restrict__ state_slots, const float* __restrict__ norm_w,
                 void* out, int out_dtype, int H, int N, int P, float q_scale, float eps, int in_smem) {
   using V = typename Cols<VEC>::T;
-  extern __shared__ __align__(16) float gs_smem[];   // q [N], k [N], alpha [N], v [P], o [P], shares [RG][P], state [N][P] (in_smem)
+  extern __shared__ __align__(16) float gs_smem[];   // q [N], k [N], alpha [N], v [P], o [P], hidden [R], shares [RG][P], state [N][P] (in_smem)
   __shared__ float scratch[32];
-  pdl_prologue(proj.p, log_decay, state);
+  pdl_prologue(proj.p, dec.hidden.p, state);
   const int b = blockIdx.x, h = blockIdx.y;
   const int t0 = cu_q_lens[b], n_tok = cu_q_lens[b + 1] - t0;
   if (n_tok <= 0) return;
@@ -110,7 +92,8 @@ gla_step_kernel(Source proj, long long row_width, const float* log_decay, float*
   float* as = ks + np;
   float* vs = as + np;
   float* os = vs + pp;
-  float* part = os + pp;
+  float* hs = os + pp;
+  float* part = hs + (dec.R + 3) / 4 * 4;
   const int cols = P / VEC;
   const int CG = cols < ST ? cols : ST, RG = ST / CG;
   const int cg = threadIdx.x % CG, rg = threadIdx.x / CG;
@@ -132,12 +115,20 @@ gla_step_kernel(Source proj, long long row_width, const float* log_decay, float*
   for (int k = 0; k < n_tok; ++k) {
     const int t = t0 + k;
     const long long row = (long long)t * row_width;
-    for (int i = threadIdx.x; i < 3 * N; i += ST) {
+    for (int i = threadIdx.x; i < dec.R; i += ST) hs[i] = source_load(dec.hidden, (long long)t * dec.row_width + dec.at + i);
+    for (int i = threadIdx.x; i < 2 * N; i += ST) {
       if (i < N) qs[i] = __fmul_rn(load(row + qc + i), q_scale);
-      else if (i < 2 * N) ks[i - N] = load(row + kc + i - N);
-      else as[i - 2 * N] = expf(log_decay[((long long)t * H + h) * N + i - 2 * N]);
+      else ks[i - N] = load(row + kc + i - N);
     }
     for (int i = threadIdx.x; i < P; i += ST) vs[i] = load(row + vc + i);
+    __syncthreads();
+    for (int i = threadIdx.x; i < N; i += ST) {
+      float z = 0.f;
+#pragma unroll 8
+      for (int r = 0; r < dec.R; ++r)
+        z = __fmaf_rn(hs[r], load_as(dec.a2_t, dec.dtype, (long long)r * H * N + (long long)h * N + i), z);
+      as[i] = expf(log_decay(z, dec.bias[h * N + i], dec.tau));
+    }
     __syncthreads();
     if (rg < RG)
       for (int c = cg; c < cols; c += CG) {
@@ -187,10 +178,10 @@ gla_step_kernel(Source proj, long long row_width, const float* log_decay, float*
 // planes: q hi, q lo, k hi, k lo, each [tokens][H N] (plane elements apart).  edges [places][H][2 RUNS][N]: M_0 ..
 // M_3, E_0 .. E_3.
 __global__ void __launch_bounds__(512)
-gla_prepare_kernel(const __nv_bfloat16* proj, long long row_width, const float* log_decay, const int* __restrict__ cu,
-                   int B, int t_first, __nv_bfloat16* planes, long long plane, float* edges, int H, int N, float q_scale) {
-  extern __shared__ float2 gp_smem[];                   // the runs' own M and E [2][RUNS][N / 2]
-  pdl_prologue(proj, log_decay);
+gla_prepare_kernel(const __nv_bfloat16* proj, long long row_width, Decays dec, const int* __restrict__ cu, int B,
+                   int t_first, __nv_bfloat16* planes, long long plane, float* edges, int H, int N, float q_scale) {
+  extern __shared__ __align__(16) float gp_smem[];      // hidden [R][CH], then the runs' own M and E [2][RUNS][N]
+  pdl_prologue(proj, dec.hidden.p);
   int b, first, count;
   if (!chunk_at(cu, B, blockIdx.x, b, first, count)) return;
   const int h = blockIdx.y, half = N / 2;
@@ -205,15 +196,36 @@ gla_prepare_kernel(const __nv_bfloat16* proj, long long row_width, const float* 
     if (j0 + j < count) {
       const long long t = t0 + j0 + j;
       const __nv_bfloat16* src = proj + t * row_width + (long long)h * N + d;
-      g[j] = *reinterpret_cast<const float2*>(log_decay + (t * H + h) * N + d);
       q[j] = *reinterpret_cast<const unsigned*>(src);
       k[j] = *reinterpret_cast<const unsigned*>(src + (long long)H * N);
     }
   }
+  for (int i = threadIdx.x; i < CH * dec.R; i += blockDim.x) {
+    const int j = i / dec.R, r = i - j * dec.R;
+    gp_smem[r * CH + j] = j < count ? source_load(dec.hidden, (long long)(t0 + j) * dec.row_width + dec.at + r) : 0.f;
+  }
+  __syncthreads();
+  const __nv_bfloat16* a2 = reinterpret_cast<const __nv_bfloat16*>(dec.a2_t) + (long long)h * N + d;
+#pragma unroll 2
+  for (int r = 0; r < dec.R; ++r) {
+    const float2 w = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(a2 + (long long)r * H * N));
+    const float4* hr = reinterpret_cast<const float4*>(gp_smem + r * CH + j0);
 #pragma unroll
-  for (int j = 0; j < RUN; ++j) {                       // from log decays to their sums inside the run
-    g[j].x = fmaxf(g[j].x, LEAST);
-    g[j].y = fmaxf(g[j].y, LEAST);
+    for (int j4 = 0; j4 < RUN / 4; ++j4) {
+      const float4 x = hr[j4];
+      const float v[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        g[j4 * 4 + e].x = __fmaf_rn(v[e], w.x, g[j4 * 4 + e].x);
+        g[j4 * 4 + e].y = __fmaf_rn(v[e], w.y, g[j4 * 4 + e].y);
+      }
+    }
+  }
+  const float2 a2_bias = *reinterpret_cast<const float2*>(dec.bias + h * N + d);
+#pragma unroll
+  for (int j = 0; j < RUN; ++j) {                       // from the map's sums to log decays and their sums inside the run
+    g[j].x = j0 + j < count ? fmaxf(log_decay(g[j].x, a2_bias.x, dec.tau), LEAST) : 0.f;
+    g[j].y = j0 + j < count ? fmaxf(log_decay(g[j].y, a2_bias.y, dec.tau), LEAST) : 0.f;
     if (j > 0) {
       g[j].x = __fadd_rn(g[j].x, g[j - 1].x);
       g[j].y = __fadd_rn(g[j].y, g[j - 1].y);
@@ -235,8 +247,8 @@ gla_prepare_kernel(const __nv_bfloat16* proj, long long row_width, const float* 
     *reinterpret_cast<unsigned*>(dst + 2 * plane) = hi;
     *reinterpret_cast<unsigned*>(dst + 3 * plane) = lo;
   }
-  float2* mids = gp_smem;
-  float2* ends = gp_smem + RUNS * half;
+  float2* mids = reinterpret_cast<float2*>(gp_smem + CH * dec.R);
+  float2* ends = mids + RUNS * half;
   mids[run * half + d / 2] = mid;
   ends[run * half + d / 2] = g[RUN - 1];
   __syncthreads();
@@ -650,45 +662,36 @@ int launch_chunks(const __nv_bfloat16* planes, long long plane, const __nv_bfloa
   return DIB_OK;
 }
 
+constexpr int MOST_CHUNKED_RANK = 512;          // (the tokens' numbers lie in shared memory)
+bool decays_fit(int R, long long h_row, long long h_at, float tau) {
+  return R >= 1 && R <= 1024 && h_at >= 0 && h_at + R <= h_row && tau > 0.f;
+}
+
 }  // namespace
 
 extern "C" {
 
-// out [T][C] = log(sigmoid(z)) / tau, z = hidden a2_t + bias; hidden: R numbers at column `at` of rows row_width
-// apart; a2_t [R][C] of dtype (0 float32, 1 bfloat16).
-int dib_gla_decay(const void* hidden, int kind, int splits, long long stride, long long row_width, long long at,
-                  const void* a2_t, int dtype, const float* bias, float tau, float* out, int T, int R, int C, cudaStream_t st) {
-  if (T == 0) return DIB_OK;
-  if (R < 1 || R > 1024 || C < 1 || at < 0 || at + R > row_width || !(tau > 0.f) || ceil_div_host(T, GD) > 65535) return DIB_BAD_SIZE;
-  const Source src = make_source(hidden, kind, splits, stride);
-  const dim3 grid(ceil_div_host(C, 256), ceil_div_host(T, GD));
-  const size_t smem = sizeof(float) * GD * (size_t)R;
-  if (dtype == 0)
-    dib_launch(gla_decay_kernel<float>, grid, dim3(256), smem, st, src, row_width, at, (const float*)a2_t, bias, tau, out, T, R, C);
-  else if (dtype == 1)
-    dib_launch(gla_decay_kernel<__nv_bfloat16>, grid, dim3(256), smem, st, src, row_width, at, (const __nv_bfloat16*)a2_t,
-               bias, tau, out, T, R, C);
-  else return DIB_BAD_DTYPE;
-  DIB_CHECK_LAUNCH();
-  return DIB_OK;
-}
+// What the decays are made of: hidden holds R numbers a token at column h_at of rows h_row apart; a2_t [R][H N] of
+// a2_dtype (0 float32, 1 bfloat16; the chunked form: bfloat16), a2_bias [H N].
 
 // Tokens one by one: B sequences, whose boundaries and slots cu_q_lens and state_slots give (pointers to
 // the first of them).  in_smem 1: the state in shared memory while a sequence is walked (DIB_BAD_SIZE
 // when it does not fit); 0: in the slot.
-int dib_gla_step(const void* proj, int kind, int splits, long long stride, long long row_width, const float* log_decay,
-                 float* state, long long slot_stride, const int* cu_q_lens, const int* state_slots, const float* norm_w,
+int dib_gla_step(const void* proj, int kind, int splits, long long stride, long long row_width, const void* hidden,
+                 int h_kind, int h_splits, long long h_stride, long long h_row, long long h_at, const void* a2_t, int a2_dtype,
+                 const float* a2_bias, float tau, int R, float* state, long long slot_stride, const int* cu_q_lens, const int* state_slots, const float* norm_w,
                  void* out, int out_dtype, int B, int H, int N, int P, float q_scale, float eps, int in_smem,
                  cudaStream_t st) {
   if (B == 0) return DIB_OK;
   if (H < 1 || H > 65535 || N < 1 || N > 2048 || P < 1 || P > 4096 || row_width < 2ll * H * (N + P) ||
-      slot_stride < (long long)H * N * P)
+      slot_stride < (long long)H * N * P || !decays_fit(R, h_row, h_at, tau))
     return DIB_BAD_SIZE;
+  if (a2_dtype != 0 && a2_dtype != 1) return DIB_BAD_DTYPE;
   if (out_dtype != 0 && out_dtype != 1) return DIB_BAD_DTYPE;
   const bool v4 = P % 4 == 0 && slot_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(state) & 15) == 0;
   const int cols = v4 ? P / 4 : P, CG = cols < ST ? cols : ST, RG = ST / CG;
   const int np = (N + 3) / 4 * 4, pp = (P + 3) / 4 * 4;
-  const size_t smem = sizeof(float) * (3 * (size_t)np + 2 * (size_t)pp + (size_t)RG * pp + (in_smem ? (size_t)N * P : 0));
+  const size_t smem = sizeof(float) * (3 * (size_t)np + 2 * (size_t)pp + (size_t)((R + 3) / 4 * 4) + (size_t)RG * pp + (in_smem ? (size_t)N * P : 0));
   if (smem > MOST_SMEM) return DIB_BAD_SIZE;
   const Source src = make_source(proj, kind, splits, stride);
   static DeviceOnce once4, once1;
@@ -699,39 +702,50 @@ int dib_gla_step(const void* proj, int kind, int splits, long long stride, long 
       return DIB_LAUNCH_FAILED;
     once.mark();
   }
-  dib_launch(kern, dim3(B, H), dim3(ST), smem, st, src, row_width, log_decay, state, slot_stride, cu_q_lens, state_slots,
+  const Decays dec = {make_source(hidden, h_kind, h_splits, h_stride), h_row, h_at, a2_t, a2_dtype, a2_bias, tau, R};
+  dib_launch(kern, dim3(B, H), dim3(ST), smem, st, src, row_width, dec, state, slot_stride, cu_q_lens, state_slots,
              norm_w, out, out_dtype, H, N, P, q_scale, eps, in_smem);
   DIB_CHECK_LAUNCH();
   return DIB_OK;
 }
 
 // Whether a head's state fits in shared memory (dib_gla_step with in_smem 1), whatever the alignment.
-int dib_gla_state_fits(int N, int P) {
+int dib_gla_state_fits(int N, int P, int R) {
   const size_t pp = (P + 3) / 4 * 4, np = (N + 3) / 4 * 4;
   const int cols = P % 4 == 0 ? P / 4 : P;             // (the wider of the two forms' shares)
   const size_t shares = cols < ST ? ST / cols : 1;
-  return sizeof(float) * (3 * np + (2 + shares) * pp + (size_t)N * P) <= MOST_SMEM ? 1 : 0;
+  return sizeof(float) * (3 * np + (2 + shares) * pp + (size_t)((R + 3) / 4 * 4) + (size_t)N * P) <= MOST_SMEM ? 1 : 0;
 }
 
 // The chunked form: B sequences (cu and state_slots point at the first of them; its first token is
 // t_first of the step), `tokens` tokens.  proj bfloat16.  With places = tokens / 64 + B: planes 4 * tokens *
 // H * N bfloat16; edges places * H * 8 * N floats; sums places * H * N * P floats.
-int dib_gla_chunked(const void* proj, long long row_width, const float* log_decay, float* state, long long slot_stride,
+int dib_gla_chunked(const void* proj, long long row_width, const void* hidden, int h_kind, int h_splits, long long h_stride,
+                    long long h_row, long long h_at, const void* a2_t, const float* a2_bias, float tau, int R, float* state,
+                    long long slot_stride,
                     const int* cu, const int* state_slots, const float* norm_w, void* planes, float* edges, float* sums,
                     void* out, int B, int t_first, int tokens, int H, int N, int P, float q_scale, float eps,
                     cudaStream_t st) {
   if (B == 0 || tokens == 0) return DIB_OK;
   if (H < 1 || H > 65535 || B > 65535 || N < 16 || N > 256 || N % 16 || P < 16 || P > 256 || P % 16 ||
-      row_width < 2ll * H * (N + P) || row_width % 8 || slot_stride % 4)
+      row_width < 2ll * H * (N + P) || row_width % 8 || slot_stride % 4 || !decays_fit(R, h_row, h_at, tau) ||
+      R > MOST_CHUNKED_RANK)
     return DIB_BAD_SIZE;
-  if ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(log_decay) | reinterpret_cast<uintptr_t>(state) |
+  if ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(a2_t) | reinterpret_cast<uintptr_t>(a2_bias) | reinterpret_cast<uintptr_t>(state) |
        reinterpret_cast<uintptr_t>(planes) | reinterpret_cast<uintptr_t>(edges) | reinterpret_cast<uintptr_t>(sums) |
        reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(norm_w)) % 16 != 0)
     return DIB_BAD_ALIGN;
   const long long plane = (long long)tokens * H * N;
   const int places = tokens / CH + B;
-  dib_launch(gla_prepare_kernel, dim3(places, H), dim3(RUNS * N / 2), sizeof(float) * 2 * RUNS * N, st,
-             (const __nv_bfloat16*)proj, row_width, log_decay, cu, B, t_first, (__nv_bfloat16*)planes, plane, edges, H, N, q_scale);
+  static DeviceOnce once;
+  if (!once.done()) {
+    if (cudaFuncSetAttribute(gla_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST_SMEM) != cudaSuccess)
+      return DIB_LAUNCH_FAILED;
+    once.mark();
+  }
+  const Decays dec = {make_source(hidden, h_kind, h_splits, h_stride), h_row, h_at, a2_t, 1, a2_bias, tau, R};
+  dib_launch(gla_prepare_kernel, dim3(places, H), dim3(RUNS * N / 2), sizeof(float) * (2 * RUNS * (size_t)N + (size_t)CH * R), st,
+             (const __nv_bfloat16*)proj, row_width, dec, cu, B, t_first, (__nv_bfloat16*)planes, plane, edges, H, N, q_scale);
   DIB_CHECK_LAUNCH();
 #define DIB_GC(NPT, OUT_NPT, HALVES)                                                                                     \
   return launch_chunks<NPT, OUT_NPT, HALVES>((const __nv_bfloat16*)planes, plane, (const __nv_bfloat16*)proj, row_width, edges, norm_w, \

@@ -84,16 +84,13 @@ attn_prepare_kernel(Source proj, long long row_width, T* __restrict__ q_out, T* 
   T* dst = s < Hq ? q_out + ((long long)t * Hq + s) * D : cache + cache_at;
   const int half = rot / 2;
   const float pos = (float)positions[t];
-  for (int d = lane; d < D; d += 32) {
-    float v = x[d];
-    if (d < rot) {
-      const int i = d < half ? d : d - half;
-      const float a = __fmul_rn(pos, freq[i]);
-      const float c = __fmul_rn(amp, cosf(a)), sn = __fmul_rn(amp, sinf(a));
-      v = d < half ? __fmaf_rn(x[d], c, -__fmul_rn(x[d + half], sn)) : __fmaf_rn(x[d], c, __fmul_rn(x[d - half], sn));
-    }
-    Elem<T>::store(dst + d, v);
+  for (int d = lane; d < half; d += 32) {      // a lane takes both elements of a pair
+    const float a = __fmul_rn(pos, freq[d]);
+    const float c = __fmul_rn(amp, cosf(a)), sn = __fmul_rn(amp, sinf(a)), u = x[d], w2 = x[d + half];
+    Elem<T>::store(dst + d, __fmaf_rn(u, c, -__fmul_rn(w2, sn)));
+    Elem<T>::store(dst + d + half, __fmaf_rn(w2, c, __fmul_rn(u, sn)));
   }
+  for (int d = rot + lane; d < D; d += 32) Elem<T>::store(dst + d, x[d]);
 }
 
 // The same for a whole projection row at once: one block per token, which sees every head of q and k.
@@ -117,7 +114,7 @@ attn_prepare_row_kernel(Source proj, long long row_width, const float* __restric
                         const float* state, long long slot_stride, long long tail_at,
                         const int* __restrict__ token_seq, const int* __restrict__ cu_q_lens,
                         const int* __restrict__ state_slots, float amp) {
-  extern __shared__ float smem[];      // the row's [q | k | v] (nq + nk + nv floats), then a factor per q and k head
+  extern __shared__ float smem[];      // the row's [q | k | v] (nq + nk + nv floats), a factor per q and k head, [cos | sin]
   __shared__ float scratch[32];
   pdl_prologue(proj.p, state);
   const int t = blockIdx.x;
@@ -148,11 +145,25 @@ attn_prepare_row_kernel(Source proj, long long row_width, const float* __restric
       x[i] = acc;
     }
   } else {
-    for (int i = threadIdx.x; i < nq + nk + nv; i += ROW_THREADS) {
-      float v = source_load(proj, row + i);
-      if (bias != nullptr) v = __fadd_rn(v, bias[i]);
-      x[i] = round_to<T>(v);
+    constexpr int AT_ONCE = 8;               // elements whose loads (four splits of each) are issued together
+    const int n = nq + nk + nv;
+    for (int i0 = threadIdx.x; i0 < n; i0 += AT_ONCE * ROW_THREADS) {
+      float v[AT_ONCE];
+      source_load_strided<AT_ONCE, 4>(proj, row, i0, ROW_THREADS, n, v);
+#pragma unroll
+      for (int u = 0; u < AT_ONCE; ++u) {
+        const int i = i0 + u * ROW_THREADS;
+        if (i < n) x[i] = round_to<T>(bias != nullptr ? __fadd_rn(v[u], bias[i]) : v[u]);
+      }
     }
+  }
+  const float pos = (float)positions[t];
+  const int half = rot / 2;
+  float* cs = factor + Hq + Hkv;             // the position's cosines [half] and sines [half]
+  for (int i = threadIdx.x; i < half; i += ROW_THREADS) {
+    const float a = __fmul_rn(pos, freq[i]);
+    cs[i] = __fmul_rn(amp, cosf(a));
+    cs[half + i] = __fmul_rn(amp, sinf(a));
   }
   __syncthreads();
   if (q_w != nullptr) {
@@ -188,8 +199,6 @@ attn_prepare_row_kernel(Source proj, long long row_width, const float* __restric
       off = slot % page_size;
     }
   }
-  const float pos = (float)positions[t];
-  const int half = rot / 2;
   for (int i = threadIdx.x; i < nq + nk; i += ROW_THREADS) {
     const int s = i / D, d = i - s * D;
     float v = x[i];
@@ -197,8 +206,8 @@ attn_prepare_row_kernel(Source proj, long long row_width, const float* __restric
       // the element's partner, its frequency, and whether it is the pair's first element
       const bool first = pairs ? (d & 1) == 0 : d < half;
       const int other = pairs ? (d ^ 1) : (first ? d + half : d - half);
-      const float a = __fmul_rn(pos, freq[pairs ? d >> 1 : (first ? d : d - half)]);
-      const float c = __fmul_rn(amp, cosf(a)), sn = __fmul_rn(amp, sinf(a)), o = x[s * D + other];
+      const int f = pairs ? d >> 1 : (first ? d : d - half);
+      const float c = cs[f], sn = cs[half + f], o = x[s * D + other];
       v = first ? __fmaf_rn(v, c, -__fmul_rn(o, sn)) : __fmaf_rn(v, c, __fmul_rn(o, sn));
     }
     if (s < Hq) Elem<T>::store(q_out + (long long)t * nq + i, v);
@@ -271,22 +280,20 @@ latent_prepare_kernel(Source proj, long long row_width, T* __restrict__ q_out, T
 
 // ---- latent rows whose queries go through a latent of their own -----------------------------------
 // The projection row holds, at column q_at, a query latent of Cq elements, and at column kv_at the cached
-// latent of C elements and behind it a rotated key part of R (R may be 0).  One warp per (token, slot): slot 0
-// norms the cached latent (RMS, c_w) into the token's cache row [C + R] and rotates the key part; slot 1 norms
-// the query latent (RMS, q_w) into q_latent [T][Cq].
+// latent of C elements and behind it a rotated key part of R (R may be 0).  A block per (token, latent): the
+// first norms the cached latent (RMS, c_w) into the token's cache row [C + R] and rotates the key part; the
+// second norms the query latent (RMS, q_w) into q_latent [T][Cq].
+constexpr int LR_THREADS = 128;
 template <typename T>
-__global__ void __launch_bounds__(WARPS * 32)
+__global__ void __launch_bounds__(LR_THREADS)
 latent_rows_kernel(Source proj, long long row_width, long long q_at, int Cq, const float* __restrict__ q_w,
                    T* __restrict__ q_latent, long long kv_at, int C, int R, const float* __restrict__ c_w,
                    T* __restrict__ cache, float eps, const float* __restrict__ freq, const int* __restrict__ positions,
-                   const int* __restrict__ slot_mapping, int T_tokens, int page_size, long long num_pages, int pairs,
-                   float amp) {
+                   const int* __restrict__ slot_mapping, int page_size, long long num_pages, int pairs, float amp) {
+  __shared__ float scratch[32];
   pdl_prologue(proj.p);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const long long item = (long long)blockIdx.x * WARPS + warp;
-  if (item >= 2ll * T_tokens) return;
-  const int t = (int)(item >> 1);
-  const bool query = (item & 1) != 0;
+  const int t = blockIdx.x;
+  const bool query = blockIdx.y != 0;
   T* dst;
   if (query) {
     dst = q_latent + (long long)t * Cq;
@@ -299,31 +306,31 @@ latent_rows_kernel(Source proj, long long row_width, long long q_at, int Cq, con
   const long long src = (long long)t * row_width + (query ? q_at : kv_at);
   const int n = query ? Cq : C;
   const float* w = query ? q_w : c_w;
-  constexpr int KEEP = 16;                   // elements of a lane kept in registers (the rest is read again)
+  constexpr int KEEP = 8;                    // elements of a thread kept in registers (the rest is read again)
   float v[KEEP];
+  source_load_strided<KEEP, 4>(proj, src, threadIdx.x, LR_THREADS, n, v);
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
-    const int d = lane + 32 * i;
-    v[i] = d < n ? round_to<T>(source_load(proj, src + d)) : 0.f;
+    v[i] = round_to<T>(v[i]);
     ss = __fmaf_rn(v[i], v[i], ss);
   }
-  for (int d = lane + 32 * KEEP; d < n; d += 32) {
+  for (int d = threadIdx.x + LR_THREADS * KEEP; d < n; d += LR_THREADS) {
     const float x = round_to<T>(source_load(proj, src + d));
     ss = __fmaf_rn(x, x, ss);
   }
-  const float rstd = 1.0f / sqrtf(warp_sum(ss) / (float)n + eps);
+  const float rstd = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
-    const int d = lane + 32 * i;
+    const int d = threadIdx.x + LR_THREADS * i;
     if (d < n) Elem<T>::store(dst + d, v[i] * rstd * w[d]);
   }
-  for (int d = lane + 32 * KEEP; d < n; d += 32)
+  for (int d = threadIdx.x + LR_THREADS * KEEP; d < n; d += LR_THREADS)
     Elem<T>::store(dst + d, round_to<T>(source_load(proj, src + d)) * rstd * w[d]);
   if (query || R == 0) return;
   const float pos = (float)positions[t];
   const int half = R / 2;
-  for (int d = lane; d < R; d += 32) {
+  for (int d = threadIdx.x; d < R; d += LR_THREADS) {
     const bool first = pairs ? (d & 1) == 0 : d < half;
     const float a = __fmul_rn(pos, freq[pairs ? d >> 1 : (first ? d : d - half)]);
     const float c = __fmul_rn(amp, cosf(a)), sn = __fmul_rn(amp, sinf(a));
@@ -549,7 +556,7 @@ int dib_attn_prepare_row(const void* proj, int kind, int splits, long long strid
                         state_slots == nullptr || (taps > 1 && state == nullptr)))
     return DIB_BAD_SIZE;
   if (freq == nullptr) rot = 0;
-  const size_t smem = sizeof(float) * ((size_t)Hq * D + (size_t)Hkv * (D + Dv) + Hq + Hkv);
+  const size_t smem = sizeof(float) * ((size_t)Hq * D + (size_t)Hkv * (D + Dv) + Hq + Hkv + rot);
   if (smem > 200 * 1024) return DIB_BAD_SIZE;
   const Source src = make_source(proj, kind, splits, stride);
   static DeviceOnce once32, once16;
@@ -616,14 +623,13 @@ int dib_latent_rows(const void* proj, int kind, int splits, long long stride, lo
       q_at + Cq > row_width || kv_at + C + R > row_width || q_w == nullptr || c_w == nullptr)
     return DIB_BAD_SIZE;
   const Source src = make_source(proj, kind, splits, stride);
-  const int blocks = ceil_div_host(2ll * T, WARPS);
   if (dtype == 0)
-    dib_launch(latent_rows_kernel<float>, dim3(blocks), dim3(WARPS * 32), 0, st, src, row_width, q_at, Cq, q_w,
-               (float*)q_latent, kv_at, C, R, c_w, (float*)cache, eps, freq, positions, slot_mapping, T, page_size,
+    dib_launch(latent_rows_kernel<float>, dim3(T, 2), dim3(LR_THREADS), 0, st, src, row_width, q_at, Cq, q_w,
+               (float*)q_latent, kv_at, C, R, c_w, (float*)cache, eps, freq, positions, slot_mapping, page_size,
                num_pages, pairs, amp);
   else if (dtype == 1)
-    dib_launch(latent_rows_kernel<__nv_bfloat16>, dim3(blocks), dim3(WARPS * 32), 0, st, src, row_width, q_at, Cq, q_w,
-               (__nv_bfloat16*)q_latent, kv_at, C, R, c_w, (__nv_bfloat16*)cache, eps, freq, positions, slot_mapping, T,
+    dib_launch(latent_rows_kernel<__nv_bfloat16>, dim3(T, 2), dim3(LR_THREADS), 0, st, src, row_width, q_at, Cq, q_w,
+               (__nv_bfloat16*)q_latent, kv_at, C, R, c_w, (__nv_bfloat16*)cache, eps, freq, positions, slot_mapping,
                page_size, num_pages, pairs, amp);
   else return DIB_BAD_DTYPE;
   DIB_CHECK_LAUNCH();

@@ -37,6 +37,18 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// cap * tanh(x / cap), in units of log 2: tanh(y) = 1 - 2 / (1 + e^(2 y)), the exponential and the reciprocal on
+// the special-function unit (an absolute error of about 1e-6 of the cap)
+struct SoftCap {
+  float in, size;        // 2 log2(e) / cap * scale; cap * log2(e)
+  __device__ __forceinline__ SoftCap(float cap, float scale)
+      : in(cap > 0.f ? 2.0f * MA_LOG2E * scale / cap : 0.f), size(cap * MA_LOG2E) {}
+  __device__ __forceinline__ float operator()(float score) const {
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + ex2(score * in)));
+    return __fmaf_rn(-2.0f * size, r, size);
+  }
+};
 __device__ __forceinline__ int first_seen(int pos, int mask_kind, int mask_size) {
   if (mask_kind == 1) return pos - mask_size + 1 > 0 ? pos - mask_size + 1 : 0;
   if (mask_kind == 2) return pos > 0 ? pos / mask_size * mask_size : 0;
@@ -154,6 +166,7 @@ masked_attention_mma_kernel(const __nv_bfloat16* q, __nv_bfloat16* out, const __
   const int wpos_first = pos0 + row_base / R, wpos_last = warp_has_rows ? pos0 + wr1 / R : -1;
   const int wlo_first = first_seen(wpos_first, mask_kind, mask_size);
   const float scale_log2 = scale * MA_LOG2E;
+  const SoftCap cap(softcap, scale);
 
   float o[NV16 * 2][4];
 #pragma unroll
@@ -207,7 +220,7 @@ masked_attention_mma_kernel(const __nv_bfloat16* q, __nv_bfloat16* out, const __
           const int j = k0 + n * 8 + tig * 2 + (e & 1);
           const bool sees = j <= row_pos[h] && (j >= row_lo[h] || j < keep);
           // (softcap > 0: the scaled score passes softcap * tanh(. / softcap), float32, before the softmax)
-          const float sc = softcap > 0.f ? softcap * tanhf(s[n][e] * scale / softcap) * MA_LOG2E : s[n][e] * scale_log2;
+          const float sc = softcap > 0.f ? cap(s[n][e]) : s[n][e] * scale_log2;
           s[n][e] = sees ? sc : MA_NEG_BIG;
           mx[h] = fmaxf(mx[h], s[n][e]);
         }

@@ -426,6 +426,24 @@ __global__ void moe_combine_kernel(const float* __restrict__ per_pair, const flo
                                    int top, int W) {
   pdl_prologue(per_pair, weights, shared.p, logits.p);
   const long long n = (long long)T * W;
+  if (shared.p == nullptr && (W & 3) == 0) {
+    const int W4 = W >> 2;
+    const float4* src = reinterpret_cast<const float4*>(per_pair);
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n / 4; i += (long long)gridDim.x * blockDim.x) {
+      const long long t = i / W4, c = i - t * W4;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int j = 0; j < top; ++j) {
+        const float w = weights != nullptr ? weights[t * top + j] : weight;
+        const float4 x = src[(t * top + j) * W4 + c];
+        v.x = __fmaf_rn(w, x.x, v.x);
+        v.y = __fmaf_rn(w, x.y, v.y);
+        v.z = __fmaf_rn(w, x.z, v.z);
+        v.w = __fmaf_rn(w, x.w, v.w);
+      }
+      reinterpret_cast<float4*>(out)[i] = v;
+    }
+    return;
+  }
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const long long t = i / W, c = i - t * W;
     float v = 0.f;
@@ -466,6 +484,10 @@ int moe_product(const void* a_rows, int dtype, const int* order, int max_tiles, 
   if (max_tiles == 0) return DIB_OK;
   if (K < 1 || N < 1 || tile < 1 || tile % GC_ROWS || top < 1) return DIB_BAD_SIZE;
   if (dtype == 1 && K % 8 == 0 && (tile == 16 || tile == 64)) {
+    // (few rows: narrower CTAs where those of 128 weight rows would not fill the SMs twice)
+    const long long weight_rows = mode == 0 ? 2ll * N : N;
+    if (tile == 16 && (weight_rows + 127) / 128 * max_tiles < 2 * 148 * 4)
+      return launch_product_mma<1, 2>(a_rows, order, max_tiles, tile, top, w, out, K, N, mode, limit, alpha, st);
     if (tile == 16) return launch_product_mma<1, 4>(a_rows, order, max_tiles, tile, top, w, out, K, N, mode, limit, alpha, st);
     return launch_product_mma<4, 4>(a_rows, order, max_tiles, tile, top, w, out, K, N, mode, limit, alpha, st);
   }

@@ -261,48 +261,86 @@ struct StreamTerms {
   int n;
 };
 
+// block_sum of several values at once (each in block_sum's order); scratch holds 32 floats a value
+__device__ __forceinline__ void block_sums(float (&v)[STREAM_TERMS], float* scratch) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+#pragma unroll
+  for (int k = 0; k < STREAM_TERMS; ++k) v[k] = warp_sum(v[k]);
+  __syncthreads();
+  if (lane == 0) {
+#pragma unroll
+    for (int k = 0; k < STREAM_TERMS; ++k) scratch[k * 32 + warp] = v[k];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < STREAM_TERMS; ++k) {
+    float total = 0.f;
+    for (int w = 0; w < nwarps; ++w) total += scratch[k * 32 + w];
+    v[k] = total;
+  }
+}
+
 template <int VPT, int AHEAD>
 __global__ void stream_terms_kernel(float* stream, StreamTerms terms, int norm_kind, const float* w, void* out,
                                     int out_dtype, int W, float eps) {
-  __shared__ float scratch[32];
+  __shared__ float scratch[32 * STREAM_TERMS];
   pdl_prologue(stream, terms.t[0].x.p, terms.t[1].x.p, terms.t[2].x.p);
   const long long base = (long long)blockIdx.x * W;
   const float width = (float)W;
   if (VPT > 0) {
     constexpr int N = VPT > 0 ? VPT : 1;
-    float r[N], sum[N], v[N];
+    float r[N], v[STREAM_TERMS][N], f[STREAM_TERMS];
+    // every term's loads before the first is used
 #pragma unroll
     for (int i = 0; i < N; ++i) {
       const int c = threadIdx.x + i * blockDim.x;
       r[i] = c < W ? stream[base + c] : 0.f;
-      sum[i] = 0.f;
     }
 #pragma unroll
+    for (int k = 0; k < STREAM_TERMS; ++k)
+      if (k < terms.n) source_load_strided<N, AHEAD>(terms.t[k].x, base, threadIdx.x, blockDim.x, W, v[k]);
+    bool any = false;
+#pragma unroll
     for (int k = 0; k < STREAM_TERMS; ++k) {
-      if (k >= terms.n) break;
+      f[k] = 0.f;                           // a normed term's squares, then its factor
+      if (k >= terms.n) continue;
       const StreamTerm& t = terms.t[k];
-      source_load_strided<N, AHEAD>(t.x, base, threadIdx.x, blockDim.x, W, v);
       if (t.bias != nullptr) {
 #pragma unroll
         for (int i = 0; i < N; ++i) {
           const int c = threadIdx.x + i * blockDim.x;
-          if (c < W) v[i] = __fadd_rn(v[i], t.bias[c]);
+          if (c < W) v[k][i] = __fadd_rn(v[k][i], t.bias[c]);
         }
       }
       if (t.w != nullptr) {
-        float ss = 0.f;
+        any = true;
 #pragma unroll
-        for (int i = 0; i < N; ++i) ss = __fmaf_rn(v[i], v[i], ss);
-        const float f = 1.0f / sqrtf(block_sum(ss, scratch) / width + t.eps);
+        for (int i = 0; i < N; ++i) f[k] = __fmaf_rn(v[k][i], v[k][i], f[k]);
+      }
+    }
+    if (any) {
+      block_sums(f, scratch);
+#pragma unroll
+      for (int k = 0; k < STREAM_TERMS; ++k) {
+        if (k >= terms.n || terms.t[k].w == nullptr) continue;
+        const StreamTerm& t = terms.t[k];
+        const float rs = 1.0f / sqrtf(f[k] / width + t.eps);
 #pragma unroll
         for (int i = 0; i < N; ++i) {
           const int c = threadIdx.x + i * blockDim.x;
-          if (c < W) v[i] = __fmul_rn(__fmul_rn(v[i], f), t.w[c]);
+          if (c < W) v[k][i] = __fmul_rn(__fmul_rn(v[k][i], rs), t.w[c]);
         }
       }
-#pragma unroll
-      for (int i = 0; i < N; ++i) sum[i] = __fmaf_rn(t.a, v[i], sum[i]);
     }
+    float sum[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) sum[i] = 0.f;
+#pragma unroll
+    for (int k = 0; k < STREAM_TERMS; ++k)
+      if (k < terms.n) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) sum[i] = __fmaf_rn(terms.t[k].a, v[k][i], sum[i]);
+      }
     float first = 0.f;                      // the row's sum (layer norm) or its squares' (RMS norm)
 #pragma unroll
     for (int i = 0; i < N; ++i) {

@@ -1444,30 +1444,28 @@ def gated_linear_attention(proj, hidden, hidden_col: int, a2_t: torch.Tensor, a2
                           f"of {d}/{e}")
     lib = _lib("gated_linear_attention")
     dev = state.device
-    log_decay = torch.empty(t, h * d, dtype=torch.float32, device=dev)
-    st = lib.dib_gla_decay(*_source_args(hidden), c_longlong(hidden.shape[1]), c_longlong(hidden_col), _ptr(a2_t),
-                           c_int(_dt(a2_t, "a2_t")), _ptr(a2_bias), c_float(tau), _ptr(log_decay), c_int(t), c_int(rank),
-                           c_int(h * d), _stream())
-    _check(st, "gated_linear_attention(decays)", f"a map of rank {rank} (at most 1024)")
     out = torch.empty(t, h * e, dtype=out_dtype, device=dev)
     n, nd = step.num_seqs, min(int(step.num_decode or 0), step.num_seqs)
     chunked = GLA_CHUNKED and out_dtype == torch.bfloat16 and d % 16 == 0 and e % 16 == 0 and d <= 256 and e <= 256 \
-        and width % 8 == 0
+        and width % 8 == 0 and rank <= 512 and a2_t.dtype == torch.bfloat16
+    decays = (*_source_args(hidden), c_longlong(hidden.shape[1]), c_longlong(hidden_col), _ptr(a2_t))
+    decays_tail = (_ptr(a2_bias), c_float(tau), c_int(rank))
     q_scale = float(d) ** -0.5
     stride = c_longlong(state.shape[1])
 
     def by_token(first, count, in_smem):
-        st = lib.dib_gla_step(*_source_args(proj), c_longlong(width), _ptr(log_decay), _ptr(state), stride,
+        st = lib.dib_gla_step(*_source_args(proj), c_longlong(width), *decays, c_int(_dt(a2_t, "a2_t")), *decays_tail,
+                              _ptr(state), stride,
                               c_void_p(step.cu_q_lens.data_ptr() + 4 * first),
                               c_void_p(step.state_slots.data_ptr() + 4 * first), _ptr(norm_weight), _ptr(out),
                               c_int(_DT[out_dtype]), c_int(count), c_int(h), c_int(d), c_int(e), c_float(q_scale),
                               c_float(norm_eps), c_int(in_smem), _stream())
-        _check(st, "gated_linear_attention(token by token)", f"heads of {d}/{e}")
+        _check(st, "gated_linear_attention(token by token)", f"heads of {d}/{e}, a map of rank {rank} (at most 1024)")
 
     if nd:
         by_token(0, nd, 0)
     if nd < n and not chunked:
-        by_token(nd, n - nd, int(lib.dib_gla_state_fits(c_int(d), c_int(e))))
+        by_token(nd, n - nd, int(lib.dib_gla_state_fits(c_int(d), c_int(e), c_int(rank))))
     elif nd < n:
         if isinstance(proj, SplitSum) or proj.dtype != torch.bfloat16:      # the stored bfloat16 matrix
             parts = proj.parts if isinstance(proj, SplitSum) else as_tensor(proj).unsqueeze(0)
@@ -1477,7 +1475,7 @@ def gated_linear_attention(proj, hidden, hidden_col: int, a2_t: torch.Tensor, a2
         planes = torch.empty(4, tokens, h * d, dtype=torch.bfloat16, device=dev)
         edges = torch.empty(places, h, 8, d, dtype=torch.float32, device=dev)
         sums = torch.empty(places, h, d, e, dtype=torch.float32, device=dev)
-        st = lib.dib_gla_chunked(_ptr(proj), c_longlong(width), _ptr(log_decay), _ptr(state), stride,
+        st = lib.dib_gla_chunked(_ptr(proj), c_longlong(width), *decays, *decays_tail, _ptr(state), stride,
                                  c_void_p(step.cu_q_lens.data_ptr() + 4 * nd),
                                  c_void_p(step.state_slots.data_ptr() + 4 * nd), _ptr(norm_weight), _ptr(planes),
                                  _ptr(edges), _ptr(sums), _ptr(out), c_int(n - nd), c_int(nd), c_int(tokens), c_int(h),
