@@ -484,10 +484,6 @@ int moe_product(const void* a_rows, int dtype, const int* order, int max_tiles, 
   if (max_tiles == 0) return DIB_OK;
   if (K < 1 || N < 1 || tile < 1 || tile % GC_ROWS || top < 1) return DIB_BAD_SIZE;
   if (dtype == 1 && K % 8 == 0 && (tile == 16 || tile == 64)) {
-    // (few rows: narrower CTAs where those of 128 weight rows would not fill the SMs twice)
-    const long long weight_rows = mode == 0 ? 2ll * N : N;
-    if (tile == 16 && (weight_rows + 127) / 128 * max_tiles < 2 * 148 * 4)
-      return launch_product_mma<1, 2>(a_rows, order, max_tiles, tile, top, w, out, K, N, mode, limit, alpha, st);
     if (tile == 16) return launch_product_mma<1, 4>(a_rows, order, max_tiles, tile, top, w, out, K, N, mode, limit, alpha, st);
     return launch_product_mma<4, 4>(a_rows, order, max_tiles, tile, top, w, out, K, N, mode, limit, alpha, st);
   }
